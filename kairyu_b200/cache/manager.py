@@ -3,11 +3,12 @@
 Host-side only; the tensors live in :mod:`kairyu_b200.cache.storage`.
 
 Cache slots (one per schedule call that writes a cache) with equal page
-geometry and window form a *group*; each group has its own page pool and its
+geometry, window and kept first tokens form a *group*; each group has its own page pool and its
 own block table per request, because a group that keeps every key and a group
 that keeps a window of them fill and empty at different rates.  A request's
 table for a group maps page index ``position // page_size`` to a physical page,
-or -1 once a windowed group has given the page back.
+or -1 once a windowed group has given the page back (the pages of the first tokens a
+window keeps stay for as long as the request lives).
 
 The reference's dense pool is uniform (one table per request,
 kairyu/engine/core/radix_kv.py:144-149); groups generalise it the way its
@@ -80,7 +81,7 @@ class RequestCache:
     request_id: Hashable
     state_slot: int
     tables: list[list[int]]  # per group: page index -> physical page or -1
-    first_live: list[int]  # per group: lowest page index still held
+    first_live: list[int]  # per group: lowest page index still held behind the pages of kept first tokens
     num_tokens: int = 0  # positions [0, num_tokens) have been computed
     shared: list[PrefixNode] = field(default_factory=list)  # the leading pages it reads from the prefix tree
     num_cached_tokens: int = 0  # how many tokens admission found in the tree
@@ -147,34 +148,41 @@ class CacheManager:
         return -(-num_tokens // self.page_size)
 
     def _first_needed_page(self, group: CacheGroup, query_start: int) -> int:
-        """Lowest page index a query at ``query_start`` (or later) can read."""
+        """Lowest page index a query at ``query_start`` (or later) can read through its window (the pages
+        of kept first tokens aside)."""
         if group.spec.window is None:
             return 0
         return max(0, query_start - group.spec.window + 1) // self.page_size
+
+    def kept_pages(self, group: CacheGroup) -> int:
+        """How many leading pages hold first tokens that a window keeps."""
+        return self.pages_for(group.spec.keep_first) if group.spec.window is not None else 0
+
+    def _readable_pages(self, group: CacheGroup, query_start: int, last: int) -> list[int]:
+        """Indices below ``last`` of the pages that queries from ``query_start`` on can read or write."""
+        first = self._first_needed_page(group, query_start)
+        return [*range(min(self.kept_pages(group), first, last)), *range(first, last)]
 
     def pages_needed(self, request_id: Optional[Hashable], upto: int, query_start: int) -> list[int]:
         """New pages per group to cover positions [.., upto) for queries from ``query_start``."""
         needed = []
         record = self._requests.get(request_id) if request_id is not None else None
         for group in self.layout.groups:
-            first = self._first_needed_page(group, query_start)
-            last = self.pages_for(upto)
-            if record is None:
-                needed.append(max(0, last - first))
-            else:
-                table = record.tables[group.index]
-                held = sum(1 for index in range(first, min(last, len(table))) if table[index] >= 0)
-                needed.append(max(0, last - first) - held)
+            indices = self._readable_pages(group, query_start, self.pages_for(upto))
+            table = record.tables[group.index] if record is not None else []
+            needed.append(sum(1 for index in indices if index >= len(table) or table[index] < 0))
         return needed
 
     def peak_pages(self, num_tokens: int, portion: int = 1) -> list[int]:
         """Per group, the most pages a request of ``num_tokens`` tokens holds at any time when it is
         fed in portions of at most ``portion`` tokens.  A group that keeps every key holds them all;
         a windowed group holds the window behind the portion's first query plus the portion itself
-        (one page more for a window that does not start on a page's edge)."""
+        (one page more for a window that does not start on a page's edge) and the pages of the first
+        tokens it keeps."""
         whole = self.pages_for(num_tokens)
         return [
-            whole if group.spec.window is None else min(whole, self.pages_for(group.spec.window + max(portion, 1)) + 1)
+            whole if group.spec.window is None
+            else min(whole, self.pages_for(group.spec.window + max(portion, 1)) + 1 + self.kept_pages(group))
             for group in self.layout.groups
         ]
 
@@ -242,10 +250,9 @@ class CacheManager:
             self._take_back(short)
         for group, pool in zip(self.layout.groups, self.pools):
             table = record.tables[group.index]
-            first = self._first_needed_page(group, query_start)
             while len(table) < last:
                 table.append(-1)
-            for index in range(first, last):
+            for index in self._readable_pages(group, query_start, last):
                 if table[index] < 0:
                     table[index] = pool.allocate(1)[0]
         return True
@@ -263,7 +270,7 @@ class CacheManager:
             table = record.tables[group.index]
             keep_from = self._first_needed_page(group, num_tokens)
             stale = []
-            for index in range(record.first_live[group.index], min(keep_from, len(table))):
+            for index in range(max(record.first_live[group.index], self.kept_pages(group)), min(keep_from, len(table))):
                 if table[index] >= 0:
                     stale.append(table[index])
                     table[index] = -1

@@ -6,20 +6,21 @@
 // the write of a step's keys and values into their pages.
 //
 //   q      [tokens, Hq * MAPS * D]        head by head, a head's maps side by side
-//   keys   [pages, page_size, Hkv, MAPS * D]    the same layout per key/value head
+//   keys   [pages, page_size, Hk, MAPS * D]     the same layout per key head (as many as value heads, or fewer)
 //   values [pages, page_size, Hkv, DV]
 //   s_m(i, j) = cap * tanh(q_m(i) . k_m(j) * scale / cap)      (cap <= 0: no cap)
-//   a_m(i) = sum_j softmax_j(s_m(i, j)) v(j)   over max(0, i + 1 - window) <= j <= i
+//   a_m(i) = sum_j softmax_j(s_m(i, j)) v(j)   over max(0, i + 1 - window) <= j <= i, and with a window also over j < keep_first
 //   o = a_1 - lambda * a_2   (MAPS = 1: o = a_1);  head_norm: o <- o * rsqrt(mean(o^2) + eps) * out_scale
 //   sinks (optional, one fp32 logit a query head): every map's denominator also holds exp(sink_h); a sink
 //   is a term exp(sink) of the denominator alone, taken as stored (all zeros: "one added to the denominator")
 //   gate (optional, [tokens, Hq * DV], the activations' dtype): o <- o * sigmoid(gate), last of all
 //
-// Query head h reads key/value head h / (Hq / Hkv).  The order of every sum depends on the
-// query's position, the window and the sizes only: warp w of a block takes keys start + w,
-// start + w + WARPS, ... with an online softmax of its own per map, and the warps' partial results
-// are merged in warp order.  So a token's output does not depend on what else is in the batch
-// or on how the prompt was cut.
+// Query head h reads value head h / (Hq / Hkv) and key head h / (Hq / Hk); Hk is Hkv unless the caller says that a position's
+// keys are fewer, wider rows (one row that all heads share: heads whose queries span every key/value head's key).
+// The order of every sum depends on the query's position, the window and the sizes only: of the keys a query sees, in
+// order, warp w of a block takes number w, w + WARPS, ... with an online softmax of its own per map, and the warps' partial
+// results are merged in warp order.  So a token's output does not depend on what else is in the batch
+// or on how the prompt was cut.  Queries of up to 256 columns a map are held in registers, wider ones in shared memory.
 #include "common.cuh"
 
 #define DA_WARPS 4
@@ -28,15 +29,16 @@
 
 __device__ __forceinline__ float soft_cap(float s, float cap, float inv_cap) { return cap > 0.0f ? cap * tanhf(s * inv_cap) : s; }
 
-template <typename T, int MAPS>
+template <typename T, int MAPS, bool WIDE>
 __global__ void __launch_bounds__(DA_WARPS * 32)
 diff_attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out, int out_stride,
                               const T* __restrict__ k_cache, const T* __restrict__ v_cache, const int* __restrict__ positions,
                               const int* __restrict__ row_ids, const int* __restrict__ block_table, int max_pages, int Hq,
-                              int Hkv, int D, int DV, int page_size, int num_pages, float scale, float cap, int window,
-                              float lambda, int head_norm, float eps, float out_scale, const float* __restrict__ sinks,
+                              int Hk, int Hkv, int D, int DV, int page_size, int num_pages, float scale, float cap, int window,
+                              int keep_first, float lambda, int head_norm, float eps, float out_scale, const float* __restrict__ sinks,
                               const T* __restrict__ gate, int gate_stride, int* flag) {
     pdl_wait();
+    extern __shared__ float wide_q[];  // WIDE: the query's MAPS * D columns
     __shared__ float sm_acc[DA_WARPS][MAPS][DA_MAX_D];
     __shared__ float sm_m[DA_WARPS][MAPS];
     __shared__ float sm_l[DA_WARPS][MAPS];
@@ -48,20 +50,27 @@ diff_attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restri
     const int lane = threadIdx.x & 31;
     const int pos = positions[t];
     const int row = row_ids[t];
-    const int kvh = h / (Hq / Hkv);
+    const int kh = h / (Hq / Hk), vh = h / (Hq / Hkv);
     const int* table = block_table + (size_t)row * max_pages;
     const int start = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
+    const int kept = min(keep_first, start);  // keys 0 .. kept - 1 are seen although the window has passed them
+    const int count = kept + pos + 1 - start;
     const float inv_cap = cap > 0.0f ? 1.0f / cap : 0.0f;
 
     float qv[MAPS][DA_MAX_K];
     const T* qp = q + (size_t)t * q_stride + (size_t)h * MAPS * D;
+    if constexpr (WIDE) {
+        for (int e = threadIdx.x; e < MAPS * D; e += DA_WARPS * 32) wide_q[e] = to_float(qp[e]);
+        __syncthreads();
+    } else {
 #pragma unroll
-    for (int m = 0; m < MAPS; ++m)
+        for (int m = 0; m < MAPS; ++m)
 #pragma unroll
-        for (int k = 0; k < DA_MAX_K; ++k) {
-            const int e = lane + 32 * k;
-            qv[m][k] = e < D ? to_float(qp[m * D + e]) : 0.0f;
-        }
+            for (int k = 0; k < DA_MAX_K; ++k) {
+                const int e = lane + 32 * k;
+                qv[m][k] = e < D ? to_float(qp[m * D + e]) : 0.0f;
+            }
+    }
 
     float big[MAPS], l[MAPS];
     float acc[MAPS][DA_MAX_K];
@@ -73,16 +82,17 @@ diff_attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restri
         for (int k = 0; k < DA_MAX_K; ++k) acc[m][k] = 0.0f;
     }
 
-    for (int j = start + warp; j <= pos; j += DA_WARPS) {
+    for (int n = warp; n < count; n += DA_WARPS) {
+        const int j = n < kept ? n : start + (n - kept);
         const int page_index = j / page_size;
         const int page = page_index < max_pages ? table[page_index] : -1;
         if (page < 0 || page >= num_pages) {
             if (lane == 0 && flag) atomicOr(flag, KB_FLAG_BAD_PAGE);
             continue;
         }
-        const size_t place = ((size_t)page * page_size + (j % page_size)) * Hkv + kvh;
-        const T* kp = k_cache + place * MAPS * D;
-        const T* vp = v_cache + place * DV;
+        const size_t place = (size_t)page * page_size + (j % page_size);
+        const T* kp = k_cache + (place * Hk + kh) * MAPS * D;
+        const T* vp = v_cache + (place * Hkv + vh) * DV;
         float vv[DA_MAX_K];
 #pragma unroll
         for (int k = 0; k < DA_MAX_K; ++k) {
@@ -92,10 +102,15 @@ diff_attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restri
 #pragma unroll
         for (int m = 0; m < MAPS; ++m) {
             float dot = 0.0f;
+            if constexpr (WIDE) {
+#pragma unroll 4
+                for (int e = lane; e < D; e += 32) dot += wide_q[m * D + e] * to_float(kp[m * D + e]);
+            } else {
 #pragma unroll
-            for (int k = 0; k < DA_MAX_K; ++k) {
-                const int e = lane + 32 * k;
-                if (e < D) dot += qv[m][k] * to_float(kp[m * D + e]);
+                for (int k = 0; k < DA_MAX_K; ++k) {
+                    const int e = lane + 32 * k;
+                    if (e < D) dot += qv[m][k] * to_float(kp[m * D + e]);
+                }
             }
             dot = soft_cap(warp_sum(dot) * scale, cap, inv_cap);
             const float m_new = fmaxf(big[m], dot);
@@ -173,25 +188,32 @@ diff_attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restri
 
 KB_EXPORT int kb_diff_attention_generic(const void* q, int q_stride, void* out, int out_stride, const void* k_cache,
                                         const void* v_cache, int is_bf16, const int* positions, const int* row_ids,
-                                        const int* block_table, int max_pages, int T, int Hq, int Hkv, int maps, int D, int DV,
-                                        int page_size, int num_pages, float scale, float cap, int window, float lambda,
+                                        const int* block_table, int max_pages, int T, int Hq, int Hk, int Hkv, int maps, int D, int DV,
+                                        int page_size, int num_pages, float scale, float cap, int window, int keep_first, float lambda,
                                         int head_norm, float eps, float out_scale, const float* sinks, const void* gate,
                                         int gate_stride, int* flag, cudaStream_t stream) {
     if (T == 0) return 0;
     if (!q || !out || !k_cache || !v_cache || !positions || !row_ids || !block_table) return KB_ERR_NULL;
-    if (D < 1 || D > DA_MAX_D || DV < 1 || DV > DA_MAX_D || maps < 1 || maps > 2) return KB_ERR_UNSUPPORTED_SIZE;
-    if (Hkv < 1 || Hq % Hkv != 0 || Hq > 65535) return KB_ERR_BAD_ARG;
+    const size_t wide = D > DA_MAX_D ? (size_t)maps * D * sizeof(float) : 0;  // the query's columns in shared memory
+    if (D < 1 || wide > 16 * 1024 || DV < 1 || DV > DA_MAX_D || maps < 1 || maps > 2) return KB_ERR_UNSUPPORTED_SIZE;
+    if (Hkv < 1 || Hq % Hkv != 0 || Hk < 1 || Hq % Hk != 0 || Hq > 65535 || keep_first < 0) return KB_ERR_BAD_ARG;
     dim3 grid(T, Hq);
-#define LAUNCH(TT, M)                                                                                                            \
-    kb_launch(diff_attention_generic_kernel<TT, M>, grid, dim3(DA_WARPS * 32), 0, stream, (const TT*)q, q_stride, (TT*)out,       \
-              out_stride, (const TT*)k_cache, (const TT*)v_cache, positions, row_ids, block_table, max_pages, Hq, Hkv, D, DV,     \
-              page_size, num_pages, scale, cap, window, lambda, head_norm, eps, out_scale, sinks, (const TT*)gate, gate_stride, flag)
+#define LAUNCH_AS(TT, M, W)                                                                                                      \
+    kb_launch(diff_attention_generic_kernel<TT, M, W>, grid, dim3(DA_WARPS * 32), wide, stream, (const TT*)q, q_stride, (TT*)out, \
+              out_stride, (const TT*)k_cache, (const TT*)v_cache, positions, row_ids, block_table, max_pages, Hq, Hk, Hkv, D, DV, \
+              page_size, num_pages, scale, cap, window, keep_first, lambda, head_norm, eps, out_scale, sinks, (const TT*)gate, gate_stride, flag)
+#define LAUNCH(TT, M)                       \
+    do {                                    \
+        if (wide) LAUNCH_AS(TT, M, true);   \
+        else LAUNCH_AS(TT, M, false);       \
+    } while (0)
     if (is_bf16) {
         if (maps == 2) LAUNCH(__nv_bfloat16, 2); else LAUNCH(__nv_bfloat16, 1);
     } else {
         if (maps == 2) LAUNCH(float, 2); else LAUNCH(float, 1);
     }
 #undef LAUNCH
+#undef LAUNCH_AS
     return kb_launch_result();
 }
 

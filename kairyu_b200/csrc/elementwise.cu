@@ -33,6 +33,53 @@ KB_EXPORT int kb_embedding(const void* table, int table_is_bf16, const int* ids,
     return kb_launch_result();
 }
 
+// ------------------------------------------------------------------ embedding with a norm of its own
+// out[t, :] = v * rsqrt(mean(v^2) + eps) * w with v = table[ids[t], :] * scale, as fp32 (w null: v itself), and the same row
+// into `origin` when that is given (a model that reads the embedding output again further up keeps a copy the residual
+// stream does not change).  An id outside [0, V) writes zeros and raises KB_FLAG_BAD_TOKEN.
+template <typename TT, typename TW>
+__global__ void embedding_norm_kernel(const TT* __restrict__ table, const int* __restrict__ ids, const TW* __restrict__ w,
+                                      float* __restrict__ out, float* __restrict__ origin, int H, int V, float scale, float eps, int* flag) {
+    pdl_wait();
+    __shared__ float scratch[32];
+    const int t = blockIdx.x;
+    const int id = ids[t];
+    const bool known = id >= 0 && id < V;
+    if (!known && threadIdx.x == 0 && flag) atomicOr(flag, KB_FLAG_BAD_TOKEN);
+    const TT* src = table + (size_t)(known ? id : 0) * H;
+    float ss = 0.0f;
+    if (w) {
+        for (int i = threadIdx.x; i < H; i += blockDim.x) {
+            const float v = to_float(src[i]) * scale;
+            ss += v * v;
+        }
+        ss = block_sum(ss, scratch);
+    }
+    const float inv = w ? rsqrtf(ss / (float)H + eps) : 1.0f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float v = known ? to_float(src[i]) * scale * inv * (w ? to_float(w[i]) : 1.0f) : 0.0f;
+        out[(size_t)t * H + i] = v;
+        if (origin) origin[(size_t)t * H + i] = v;
+    }
+}
+
+KB_EXPORT int kb_embedding_norm(const void* table, int table_is_bf16, const int* ids, const void* w, int w_is_bf16, float* out, float* origin,
+                                int T, int H, int V, float scale, float eps, int* flag, cudaStream_t stream) {
+    if (T == 0) return 0;
+    if (!table || !ids || !out) return KB_ERR_NULL;
+    const int threads = H >= 1024 ? 256 : 128;
+#define LAUNCH(TT, TW)                                                                                                                   \
+    kb_launch(embedding_norm_kernel<TT, TW>, dim3(T), dim3(threads), 0, stream, (const TT*)table, ids, (const TW*)w, out, origin, H, V, scale, \
+              eps, flag)
+    if (table_is_bf16) {
+        if (w_is_bf16) LAUNCH(__nv_bfloat16, __nv_bfloat16); else LAUNCH(__nv_bfloat16, float);
+    } else {
+        if (w_is_bf16) LAUNCH(float, __nv_bfloat16); else LAUNCH(float, float);
+    }
+#undef LAUNCH
+    return kb_launch_result();
+}
+
 // ------------------------------------------------------------------ learned positions
 // x[t, :] += table[positions[t], :] on the fp32 residual.  A position outside [0, P) adds nothing
 // and raises KB_FLAG_BAD_POS.

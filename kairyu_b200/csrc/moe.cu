@@ -10,6 +10,7 @@
 //   moe_route_scores  per token: softmax over all outputs, a correction that steers the choice only, groups of
 //                 neighbours of which the best stay, the K best that stay; weights = score * scale.  32-bit.
 //                 With `sigmoid` the scores are s = sigmoid(logit), each output by itself, instead of the softmax.
+//                 With `renormalise` the weights are the chosen s divided by their sum (+ 1e-20), times scale.
 //   moe_scale_rows  out[i] = src[token of i] * scale[pair of i]: the experts' input rows for a mixture whose router
 //                 weight multiplies an expert's INPUT (the experts are not linear, so it cannot move to the output).
 //   moe_activation  y = a * sigmoid(alpha a) * (b + shift) with a = min(gate, limit), b = clamp(up, +-limit)
@@ -23,6 +24,7 @@
 //                 written at the pair's place in `sorted`.  Plain form: A rows are those y rows, and
 //                 the result goes, in 32-bit, to row p of the output, so that the K rows of a token lie
 //                 together and whoever adds them (weighted by the router) does so in the order of k.
+//                 Ungated form: as the gated one, but an expert has no gate rows and its activation is relu(up)^2.
 //                 bfloat16 runs on mma.sync m16n8k16 with 32-bit accumulators, float32 on FMAs; the
 //                 sum over K runs in ascending order in both, whatever else the tile holds.
 //   moe_combine   out[t] = sum_k weight[t, k] * rows[at(t * K + k)]   (for callers that want plain rows; no weights: a
@@ -36,6 +38,11 @@
 #define MOE_TK 32
 #define MOE_MAX_EXPERTS 1024
 #define MOE_MAX_TOP 32
+
+// Which of an expert's two products a kernel runs, and what it does with the first one's rows.
+#define MOE_DOWN 0   // the second product: fp32 rows, a row a pair
+#define MOE_GATED 1  // the first product over gate rows and up rows, the gated unit in the epilogue
+#define MOE_RELU2 2  // the first product over up rows alone, relu(up)^2 in the epilogue
 
 template <typename TB>
 __global__ void __launch_bounds__(128)
@@ -91,6 +98,11 @@ __device__ __forceinline__ float expert_activation(float gate, float up, float l
     const float a = fminf(gate, limit);
     const float b = fminf(fmaxf(up, -limit), limit);
     return a * (1.0f / (1.0f + expf(-alpha * a))) * (b + shift);
+}
+
+__device__ __forceinline__ float relu_squared(float up) {
+    const float r = fmaxf(up, 0.0f);
+    return r * r;
 }
 
 __global__ void __launch_bounds__(1024)
@@ -172,7 +184,7 @@ template <typename T> struct MoeTile;
 template <> struct MoeTile<__nv_bfloat16> { static constexpr int LD = MOE_TK + 8; static constexpr int CHUNK = 8; };
 template <> struct MoeTile<float> { static constexpr int LD = MOE_TK + 1; static constexpr int CHUNK = 4; };
 
-template <typename T, bool GATED>
+template <typename T, int FORM>
 __global__ void __launch_bounds__(128)
 moe_grouped_kernel(const T* __restrict__ A, int lda, const int* __restrict__ sorted, int top, const T* __restrict__ W,
                    int N, int Kd, const int* __restrict__ tile_expert, const int* __restrict__ tile_first,
@@ -180,7 +192,8 @@ moe_grouped_kernel(const T* __restrict__ A, int lda, const int* __restrict__ sor
                    float shift, int real_experts, void* __restrict__ out, int vec) {
     constexpr int LD = MoeTile<T>::LD;
     constexpr int CHUNK = MoeTile<T>::CHUNK;
-    constexpr int NB = GATED ? 2 : 1;
+    constexpr bool FIRST = FORM != MOE_DOWN;
+    constexpr int NB = FORM == MOE_GATED ? 2 : 1;
     __shared__ __align__(16) T As[MOE_TM][LD];
     __shared__ __align__(16) T Bs[NB][MOE_TN][LD];
     __shared__ int a_row[MOE_TM];   // source row of A per tile row, -1: none
@@ -195,14 +208,14 @@ moe_grouped_kernel(const T* __restrict__ A, int lda, const int* __restrict__ sor
         int src = -1, dst = -1;
         if (i < rows) {
             const int p = sorted[first + i];
-            src = GATED ? p / top : first + i;
-            dst = GATED ? first + i : p;
+            src = FIRST ? p / top : first + i;
+            dst = FIRST ? first + i : p;
         }
         a_row[i] = src;
         o_row[i] = dst;
     }
     __syncthreads();
-    const size_t weight_rows = (size_t)(GATED ? 2 : 1) * N;
+    const size_t weight_rows = (size_t)NB * N;
     const T* We = W + (size_t)expert * weight_rows * Kd;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
@@ -268,9 +281,11 @@ moe_grouped_kernel(const T* __restrict__ A, int lda, const int* __restrict__ sor
                     for (int c = 0; c < 2; ++c) {
                         const int n = n0 + wn + j * 8 + 2 * tg + c;
                         if (n >= N) continue;
-                        if constexpr (GATED)
+                        if constexpr (FORM == MOE_GATED)
                             reinterpret_cast<T*>(out)[(size_t)dst * N + n] =
-                                from_float<T>(expert_activation(acc[0][i][j][half * 2 + c], acc[1][i][j][half * 2 + c], limit, alpha, shift));
+                                from_float<T>(expert_activation(acc[0][i][j][half * 2 + c], acc[NB - 1][i][j][half * 2 + c], limit, alpha, shift));
+                        else if constexpr (FORM == MOE_RELU2)
+                            reinterpret_cast<T*>(out)[(size_t)dst * N + n] = from_float<T>(relu_squared(acc[0][i][j][half * 2 + c]));
                         else
                             reinterpret_cast<float*>(out)[(size_t)dst * N + n] = acc[0][i][j][half * 2 + c];
                     }
@@ -321,8 +336,10 @@ moe_grouped_kernel(const T* __restrict__ A, int lda, const int* __restrict__ sor
             for (int j = 0; j < 8; ++j) {
                 const int n = n0 + tx + 8 * j;
                 if (n >= N) continue;
-                if constexpr (GATED)
+                if constexpr (FORM == MOE_GATED)
                     reinterpret_cast<T*>(out)[(size_t)dst * N + n] = from_float<T>(expert_activation(acc[0][i][j], acc[NB - 1][i][j], limit, alpha, shift));
+                else if constexpr (FORM == MOE_RELU2)
+                    reinterpret_cast<T*>(out)[(size_t)dst * N + n] = from_float<T>(relu_squared(acc[0][i][j]));
                 else
                     reinterpret_cast<float*>(out)[(size_t)dst * N + n] = acc[0][i][j];
             }
@@ -341,7 +358,7 @@ moe_grouped_kernel(const T* __restrict__ A, int lda, const int* __restrict__ sor
 #define SK_PAIRS 8
 #define SK_FEATURES 64
 
-template <bool GATED>
+template <int FORM>
 __global__ void __launch_bounds__(128)
 moe_skinny_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int* __restrict__ sorted, int top,
                   const __nv_bfloat16* __restrict__ W, int N, int Kd, int Kp, const int* __restrict__ tile_expert,
@@ -349,7 +366,8 @@ moe_skinny_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int* __res
                   float limit, float alpha, float shift, int real_experts, void* __restrict__ out) {
     extern __shared__ __align__(16) unsigned char sk_shared[];
     __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(sk_shared);  // [SK_PAIRS][Kp + 32]
-    constexpr int NB = GATED ? 2 : 1;
+    constexpr bool FIRST = FORM != MOE_DOWN;
+    constexpr int NB = FORM == MOE_GATED ? 2 : 1;
     const int ldx = Kp + 32;  // rows fall on alternate halves of a 128-byte line: 16-byte reads of 8 rows do not collide
     pdl_wait();
     const int tile = blockIdx.x;
@@ -378,7 +396,7 @@ moe_skinny_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int* __res
             uint4 v = zero4;
             if (i < np && c < Kd) {
                 const int place = first + sub + i;
-                const int src = GATED ? sorted[place] / top : place;
+                const int src = FIRST ? sorted[place] / top : place;
                 v = *reinterpret_cast<const uint4*>(A + (size_t)src * lda + c);
             }
             *reinterpret_cast<uint4*>(xs + (size_t)i * ldx + c) = v;
@@ -433,9 +451,11 @@ moe_skinny_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int* __res
             const int i = 2 * tg + (c & 1);
             if (feature >= N || i >= np) continue;
             const int place = first + sub + i;
-            if constexpr (GATED)
+            if constexpr (FORM == MOE_GATED)
                 reinterpret_cast<__nv_bfloat16*>(out)[(size_t)place * N + feature] =
                     __float2bfloat16_rn(expert_activation(acc[0][c], acc[NB - 1][c], limit, alpha, shift));
+            else if constexpr (FORM == MOE_RELU2)
+                reinterpret_cast<__nv_bfloat16*>(out)[(size_t)place * N + feature] = __float2bfloat16_rn(relu_squared(acc[0][c]));
             else
                 reinterpret_cast<float*>(out)[(size_t)sorted[place] * N + feature] = acc[0][c];
         }
@@ -498,7 +518,7 @@ KB_EXPORT int kb_moe_scale_rows(const void* src, int is_bf16, const int* rows, i
 template <typename TB>
 __global__ void __launch_bounds__(128)
 moe_route_scores_kernel(const float* __restrict__ logits, const TB* __restrict__ correction, int n, int K, int groups, int keep,
-                        float scale, int sigmoid, int stride, int* __restrict__ ids, float* __restrict__ weights, int T) {
+                        float scale, int sigmoid, int renormalise, int stride, int* __restrict__ ids, float* __restrict__ weights, int T) {
     extern __shared__ float route_shared[];  // per warp: s[n], c[n], group values [groups]
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -541,7 +561,7 @@ moe_route_scores_kernel(const float* __restrict__ logits, const TB* __restrict__
         }
         __syncwarp();
     }
-    float last_value = INFINITY;
+    float last_value = INFINITY, chosen_sum = 0.0f;
     int last_id = -1;
     for (int k = 0; k < K; ++k) {
         float best = -INFINITY;
@@ -568,13 +588,18 @@ moe_route_scores_kernel(const float* __restrict__ logits, const TB* __restrict__
             ids[(size_t)t * K + k] = best_id;
             weights[(size_t)t * K + k] = s[best_id] * scale;
         }
+        chosen_sum += s[best_id];
         last_value = best;
         last_id = best_id;
+    }
+    if (renormalise) {
+        __syncwarp();
+        for (int k = lane; k < K; k += 32) weights[(size_t)t * K + k] /= chosen_sum + 1e-20f;
     }
 }
 
 KB_EXPORT int kb_moe_route_scores(const float* logits, const void* correction, int correction_is_bf16, int n, int K, int groups,
-                                  int keep, float scale, int sigmoid, int stride, int* ids, float* weights, int T, cudaStream_t stream) {
+                                  int keep, float scale, int sigmoid, int renormalise, int stride, int* ids, float* weights, int T, cudaStream_t stream) {
     if (T == 0) return 0;
     if (!logits || !ids || !weights) return KB_ERR_NULL;
     if (n < 1 || K < 1 || K > n || n > MOE_MAX_EXPERTS) return KB_ERR_UNSUPPORTED_SIZE;
@@ -583,10 +608,10 @@ KB_EXPORT int kb_moe_route_scores(const float* logits, const void* correction, i
     if (smem > 48 * 1024) return KB_ERR_UNSUPPORTED_SIZE;
     if (correction_is_bf16)
         kb_launch(moe_route_scores_kernel<__nv_bfloat16>, dim3((T + 3) / 4), dim3(128), smem, stream, logits, (const __nv_bfloat16*)correction,
-                  n, K, groups, keep, scale, sigmoid, stride, ids, weights, T);
+                  n, K, groups, keep, scale, sigmoid, renormalise, stride, ids, weights, T);
     else
         kb_launch(moe_route_scores_kernel<float>, dim3((T + 3) / 4), dim3(128), smem, stream, logits, (const float*)correction, n, K, groups,
-                  keep, scale, sigmoid, stride, ids, weights, T);
+                  keep, scale, sigmoid, renormalise, stride, ids, weights, T);
     return kb_launch_result();
 }
 
@@ -628,7 +653,7 @@ KB_EXPORT int kb_moe_activation(const void* gate_up, void* y, int is_bf16, int r
 }
 
 KB_EXPORT int kb_moe_grouped(const void* A, int lda, const int* sorted, int top, const void* W, int N, int Kd, int is_bf16,
-                             int gated, const int* tile_expert, const int* tile_first, const int* tile_pairs,
+                             int form, const int* tile_expert, const int* tile_first, const int* tile_pairs,
                              const int* num_tiles, int max_tiles, float limit, float alpha, float shift, int real_experts, void* out,
                              cudaStream_t stream) {
     if (max_tiles == 0) return 0;
@@ -641,15 +666,15 @@ KB_EXPORT int kb_moe_grouped(const void* A, int lda, const int* sorted, int top,
     kb_launch(moe_grouped_kernel<T, G>, grid, dim3(128), 0, stream, (const T*)A, lda, sorted, top, (const T*)W, N, Kd, tile_expert, \
               tile_first, tile_pairs, num_tiles, limit, alpha, shift, real_experts, out, vec)
     if (is_bf16) {
-        if (gated) LAUNCH(__nv_bfloat16, true); else LAUNCH(__nv_bfloat16, false);
+        if (form == MOE_GATED) LAUNCH(__nv_bfloat16, MOE_GATED); else if (form == MOE_RELU2) LAUNCH(__nv_bfloat16, MOE_RELU2); else LAUNCH(__nv_bfloat16, MOE_DOWN);
     } else {
-        if (gated) LAUNCH(float, true); else LAUNCH(float, false);
+        if (form == MOE_GATED) LAUNCH(float, MOE_GATED); else if (form == MOE_RELU2) LAUNCH(float, MOE_RELU2); else LAUNCH(float, MOE_DOWN);
     }
 #undef LAUNCH
     return kb_launch_result();
 }
 
-KB_EXPORT int kb_moe_skinny(const void* A, int lda, const int* sorted, int top, const void* W, int N, int Kd, int gated,
+KB_EXPORT int kb_moe_skinny(const void* A, int lda, const int* sorted, int top, const void* W, int N, int Kd, int form,
                             const int* tile_expert, const int* tile_first, const int* tile_pairs, const int* num_tiles,
                             int max_tiles, float limit, float alpha, float shift, int real_experts, void* out, cudaStream_t stream) {
     if (max_tiles == 0) return 0;
@@ -659,15 +684,16 @@ KB_EXPORT int kb_moe_skinny(const void* A, int lda, const int* sorted, int top, 
     const size_t smem = (size_t)SK_PAIRS * (Kp + 32) * sizeof(__nv_bfloat16);
     if (smem > 200 * 1024) return KB_ERR_UNSUPPORTED_SIZE;
     dim3 grid(max_tiles, (N + SK_FEATURES - 1) / SK_FEATURES);
-    if (gated) {
-        if (smem > 48 * 1024) cudaFuncSetAttribute(moe_skinny_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        kb_launch(moe_skinny_kernel<true>, grid, dim3(128), smem, stream, (const __nv_bfloat16*)A, lda, sorted, top, (const __nv_bfloat16*)W, N, Kd, Kp,
-                  tile_expert, tile_first, tile_pairs, num_tiles, limit, alpha, shift, real_experts, out);
-    } else {
-        if (smem > 48 * 1024) cudaFuncSetAttribute(moe_skinny_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        kb_launch(moe_skinny_kernel<false>, grid, dim3(128), smem, stream, (const __nv_bfloat16*)A, lda, sorted, top, (const __nv_bfloat16*)W, N, Kd, Kp,
-                  tile_expert, tile_first, tile_pairs, num_tiles, limit, alpha, shift, real_experts, out);
-    }
+#define LAUNCH(F)                                                                                                                             \
+    do {                                                                                                                                      \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(moe_skinny_kernel<F>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);               \
+        kb_launch(moe_skinny_kernel<F>, grid, dim3(128), smem, stream, (const __nv_bfloat16*)A, lda, sorted, top, (const __nv_bfloat16*)W, N, Kd, \
+                  Kp, tile_expert, tile_first, tile_pairs, num_tiles, limit, alpha, shift, real_experts, out);                                  \
+    } while (0)
+    if (form == MOE_GATED) LAUNCH(MOE_GATED);
+    else if (form == MOE_RELU2) LAUNCH(MOE_RELU2);
+    else LAUNCH(MOE_DOWN);
+#undef LAUNCH
     return kb_launch_result();
 }
 

@@ -218,7 +218,7 @@ class ModelRunner:
                 first = 0
                 if group.spec.window is not None:  # pages the window has passed may be gone
                     first = max(0, (seq_len - len(entry.tokens) + 1 - group.spec.window)) // page_size
-                for index in range(first, needed):
+                for index in [*range(min(self.cache.kept_pages(group), first)), *range(first, needed)]:
                     page = table[index]
                     if page <= 0 or page >= self.cache.num_pages:
                         raise StepError(f"request {entry.request_id!r}: page {page} at place {index} of group {group.index} is not a page a request can hold")

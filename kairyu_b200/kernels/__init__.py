@@ -122,6 +122,24 @@ def embedding(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, flag: O
     _check(fn(table.data_ptr(), _is_bf16(table, "embedding"), ids.data_ptr(), out.data_ptr(), ids.numel(), H, V, float(scale), _ptr(flag), _stream()), "embedding")
 
 
+def embedding_norm(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, *, weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+                   scale: float = 1.0, origin: Optional[torch.Tensor] = None, flag: Optional[torch.Tensor] = None) -> None:
+    """out[t] = rmsnorm(table[ids[t]] * scale) * weight as fp32 (``weight=None``: no norm), and the same rows into ``origin``
+    when that is given."""
+    what = "embedding_norm"
+    _need_cuda(what, table, ids, out, weight, origin, flag)
+    _need_i32(what, ids)
+    V, H = table.shape
+    for rows in (out, origin):
+        if rows is not None and (rows.dtype != torch.float32 or rows.shape != (ids.numel(), H) or not rows.is_contiguous()):
+            raise KernelError(f"{what}: the outputs must be contiguous fp32 [tokens, hidden]")
+    if not table.is_contiguous() or (weight is not None and (weight.numel() != H or not weight.is_contiguous())):
+        raise KernelError(f"{what}: the table and the weight must be contiguous and of one width")
+    fn = _fn("elementwise", "kb_embedding_norm", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p])
+    _check(fn(table.data_ptr(), _is_bf16(table, what), ids.data_ptr(), _ptr(weight), _is_bf16(weight, what) if weight is not None else 0, out.data_ptr(),
+              _ptr(origin), ids.numel(), H, V, float(scale), float(eps), _ptr(flag), _stream()), what)
+
+
 def add_positions(table: torch.Tensor, positions: torch.Tensor, x: torch.Tensor, flag: Optional[torch.Tensor] = None) -> None:
     """x[t] += table[positions[t]] on the fp32 residual (learned absolute positions)."""
     _need_cuda("add_positions", table, positions, x, flag)
@@ -519,11 +537,11 @@ def paged_kv_write(
 
 def _check_diff_attention(what: str, q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, num_q_heads: int,
                           maps: int) -> tuple[int, int, int, int, int]:
-    num_pages, page_size, num_kv_heads, key_width = k_cache.shape
+    num_pages, page_size, num_key_heads, key_width = k_cache.shape
     if maps not in (1, 2) or key_width % maps:
         raise KernelError(f"{what}: {maps} maps over key rows of {key_width}")
-    dim, vdim = key_width // maps, v_cache.shape[3]
-    if v_cache.shape[:3] != k_cache.shape[:3] or not k_cache.is_contiguous() or not v_cache.is_contiguous():
+    dim, vdim, num_kv_heads = key_width // maps, v_cache.shape[3], v_cache.shape[2]
+    if v_cache.shape[:2] != k_cache.shape[:2] or num_q_heads % num_key_heads or not k_cache.is_contiguous() or not v_cache.is_contiguous():
         raise KernelError(f"{what}: caches must be contiguous and of one page geometry")
     if q.dtype != k_cache.dtype or out.dtype != q.dtype or v_cache.dtype != q.dtype or q.stride(1) != 1 or out.stride(1) != 1:
         raise KernelError(f"{what}: one dtype and unit inner strides")
@@ -554,6 +572,7 @@ def diff_attention_generic(
     scale: float,
     softcap: float = 0.0,
     window: int = 0,
+    keep_first: int = 0,
     lam: float = 0.0,
     head_norm_eps: Optional[float] = None,
     out_scale: float = 1.0,
@@ -565,7 +584,9 @@ def diff_attention_generic(
     arithmetic.  ``q``: [tokens, >= heads * maps * dim], a head's maps side by side; the key cache
     [pages, page, kv_heads, maps * dim] the same way; values [pages, page, kv_heads, vdim].  Scores
     q.k * scale, capped as softcap * tanh(s / softcap) when softcap > 0; a token sees itself and the
-    ``window - 1`` before it (0: all).  o = a_1 - lam * a_2; with ``head_norm_eps`` each head's o is divided
+    ``window - 1`` before it (0: all), and with a window also the sequence's first ``keep_first`` tokens.  A key cache
+    [pages, page, key_heads, ...] of fewer, wider key heads than the value cache's: query head h reads key head
+    h // (heads / key_heads) and value head h // (heads / kv_heads).  o = a_1 - lam * a_2; with ``head_norm_eps`` each head's o is divided
     by its root mean square (eps inside the root) and multiplied by ``out_scale``.  ``out``: [tokens, heads * vdim].
     ``sinks``: fp32 [heads], a logit a head that joins every map's denominator (a term exp(sink) there and nothing else).
     ``gate``: [tokens, >= heads * vdim] in the activations' dtype (a view into the packed rows is fine): the output
@@ -575,16 +596,74 @@ def diff_attention_generic(
     _check_sinks_gate(what, q, out, num_q_heads, sinks, gate)
     _need_i32(what, positions, row_ids, block_table)
     num_pages, page_size, num_kv_heads, dim, vdim = _check_diff_attention(what, q, out, k_cache, v_cache, num_q_heads, maps)
-    if dim > 256 or vdim > 256:
-        raise KernelError(f"{what}: key width {dim} or value width {vdim} > 256 is not supported")
+    if maps * dim > 4096 or vdim > 256:
+        raise KernelError(f"{what}: key rows of {maps * dim} > 4096 or values of {vdim} > 256 are not supported")
     fn = _fn("diff_attention", "kb_diff_attention_generic",
              [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-              c_int, c_int, c_int, c_float, c_float, c_int, c_float, c_int, c_float, c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p])
+              c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_float, c_int, c_float, c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p])
     _check(fn(q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), _is_bf16(q, what),
-              positions.data_ptr(), row_ids.data_ptr(), block_table.data_ptr(), block_table.shape[1], q.shape[0], num_q_heads, num_kv_heads,
-              int(maps), dim, vdim, page_size, num_pages, float(scale), float(softcap), int(window), float(lam),
-              0 if head_norm_eps is None else 1, float(head_norm_eps or 0.0), float(out_scale), _ptr(sinks), _ptr(gate),
+              positions.data_ptr(), row_ids.data_ptr(), block_table.data_ptr(), block_table.shape[1], q.shape[0], num_q_heads,
+              k_cache.shape[2], num_kv_heads, int(maps), dim, vdim, page_size, num_pages, float(scale), float(softcap), int(window), int(keep_first),
+              float(lam), 0 if head_norm_eps is None else 1, float(head_norm_eps or 0.0), float(out_scale), _ptr(sinks), _ptr(gate),
               gate.stride(0) if gate is not None else 0, _ptr(flag), _stream()), what)
+
+
+def talking_prepare(
+    packed: torch.Tensor,
+    talk: torch.Tensor,
+    mixed: torch.Tensor,
+    *,
+    num_q_heads: int,
+    num_kv_heads: int,
+    head_dim: int,
+    k_offset: int,
+    v_offset: int,
+    positions: torch.Tensor,
+    row_ids: torch.Tensor,
+    cos: Optional[torch.Tensor] = None,
+    sin: Optional[torch.Tensor] = None,
+    block_table: Optional[torch.Tensor] = None,
+    write_from: Optional[torch.Tensor] = None,
+    k_cache: Optional[torch.Tensor] = None,
+    v_cache: Optional[torch.Tensor] = None,
+    flag: Optional[torch.Tensor] = None,
+) -> None:
+    """For attention whose heads' scores are mixed before the softmax (score_h <- sum_g talk[h, g] score_g): on the packed rows
+    ``[q | ... k at k_offset ... values at v_offset ...]`` (``v_offset = k_offset``: a value is the key before its turn), the
+    first ``2 * cos.shape[1]`` columns of every head of q and k turn by the token's position, pairs (i, i + half); k and the
+    values go to their pages (if caches are given); and ``mixed`` [tokens, heads * kv_heads * dim] takes the mixed queries:
+    head h's row holds, key/value head after key/value head, sum over that head's queries g of talk[h, g] * q_g, formed in
+    32-bit.  Its product with a position's keys side by side is the mixed score.  ``talk``: fp32 [heads, heads]."""
+    what = "talking_prepare"
+    _need_cuda(what, packed, talk, mixed, positions, row_ids, cos, sin, block_table, write_from, k_cache, v_cache, flag)
+    _need_i32(what, positions, row_ids, block_table, write_from)
+    kv_width = num_kv_heads * head_dim
+    if num_q_heads % num_kv_heads or talk.dtype != torch.float32 or talk.shape != (num_q_heads, num_q_heads) or not talk.is_contiguous():
+        raise KernelError(f"{what}: heads must divide, and the mix be contiguous fp32 [heads, heads]")
+    if packed.stride(1) != 1 or mixed.stride(1) != 1 or mixed.dtype != packed.dtype or mixed.shape != (packed.shape[0], num_q_heads * kv_width) \
+            or k_offset < num_q_heads * head_dim or max(k_offset, v_offset) + kv_width > packed.shape[1] or v_offset < 0:
+        raise KernelError(f"{what}: the packed rows do not hold q, k and the values where the offsets say, or the mixed rows do not fit")
+    half = max_pos = 0
+    if cos is not None:
+        if sin is None or cos.shape != sin.shape or cos.dtype != torch.float32 or sin.dtype != torch.float32 or not (cos.is_contiguous() and sin.is_contiguous()):
+            raise KernelError(f"{what}: cos and sin must be contiguous fp32 tables of one shape")
+        max_pos, half = cos.shape
+        if 2 * half > head_dim:
+            raise KernelError(f"{what}: {2 * half} rotated columns in a head of {head_dim}")
+    page_size = num_pages = max_pages = num_rows = 0
+    if k_cache is not None:
+        if v_cache is None or block_table is None or k_cache.dtype != packed.dtype or v_cache.dtype != packed.dtype \
+                or tuple(k_cache.shape[2:]) != (num_kv_heads, head_dim) or v_cache.shape != k_cache.shape or not (k_cache.is_contiguous() and v_cache.is_contiguous()):
+            raise KernelError(f"{what}: contiguous caches of the heads' geometry in the activations' dtype, and a block table")
+        num_pages, page_size = k_cache.shape[:2]
+        num_rows, max_pages = block_table.shape
+    fn = _fn("talking_attention", "kb_talking_prepare",
+             [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p,
+              c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p])
+    _check(fn(packed.data_ptr(), packed.stride(0), _is_bf16(packed, what), packed.shape[0], int(k_offset), int(v_offset), num_q_heads, num_kv_heads,
+              head_dim, talk.data_ptr(), _ptr(cos), _ptr(sin), half, max_pos, positions.data_ptr(), row_ids.data_ptr(), _ptr(block_table), max_pages,
+              num_rows, _ptr(write_from), _ptr(k_cache), _ptr(v_cache), page_size, num_pages, mixed.data_ptr(), mixed.stride(0), _ptr(flag),
+              _stream()), what)
 
 
 DIFF_ATTENTION_TILE = 64  # queries a tile of the tensor-core kernel for prompt portions
@@ -625,7 +704,7 @@ def diff_attention_mma(
     _need_cuda(what, q, out, k_cache, v_cache, block_table, flag)
     _need_i32(what, block_table)
     num_pages, page_size, num_kv_heads, dim, vdim = _check_diff_attention(what, q, out, k_cache, v_cache, num_q_heads, maps)
-    if maps != 2 or q.dtype != torch.bfloat16 or not diff_attention_mma_supported(dim, vdim, num_q_heads, num_kv_heads):
+    if maps != 2 or q.dtype != torch.bfloat16 or k_cache.shape[2] != num_kv_heads or not diff_attention_mma_supported(dim, vdim, num_q_heads, num_kv_heads):
         raise KernelError(f"{what}: bfloat16, two maps, sizes as diff_attention_mma_supported says")
     fn = _fn("diff_attention_mma", "kb_diff_attention_mma",
              [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
@@ -1519,11 +1598,13 @@ class ResidualCopy:
 class WeightedRows:
     """A sub-layer's output as K rows a token and their weights (a mixture of experts before the
     sum): ``rows`` [tokens * K, width], ``weights`` [tokens, K] fp32; row k of token t is
-    ``rows[t * K + k]``, or ``rows[at[t * K + k]]`` where ``at`` (int32) is given."""
+    ``rows[t * K + k]``, or ``rows[at[t * K + k]]`` where ``at`` (int32) is given.  ``extra`` [tokens, width], in the
+    activation dtype: an always-on expert's rows, added after the weighted ones."""
 
     rows: torch.Tensor
     weights: torch.Tensor
     at: Optional[torch.Tensor] = None
+    extra: Optional[torch.Tensor] = None
 
 
 def output_norm_add(residual: torch.Tensor, y, weight: torch.Tensor, eps: float, copy: Optional[torch.Tensor]) -> None:
@@ -1534,6 +1615,8 @@ def output_norm_add(residual: torch.Tensor, y, weight: torch.Tensor, eps: float,
     K = 1
     rows = y
     if isinstance(y, WeightedRows):
+        if y.extra is not None:
+            raise KernelError("output_norm_add: weighted rows with an always-on expert's rows are added by their own kernel")
         rows, mix, at = y.rows, y.weights, y.at
         K = mix.shape[1]
         _need_i32("output_norm_add", at)
@@ -1554,6 +1637,58 @@ def output_norm_add(residual: torch.Tensor, y, weight: torch.Tensor, eps: float,
            float(eps), _stream()),
         "output_norm_add",
     )
+
+
+@dataclass
+class PendingGated:
+    """What a block whose sub-layers' results are gated element by element leaves for the norm that reads the stream next:
+    ``residual += mult * sigmoid(gate + bias) * values`` is still to be done, and that norm's kernel does it on its way.
+    ``values``: rows of the residual's shape, or a :class:`WeightedRows` (a mixture before its sum)."""
+
+    values: object
+    gate: torch.Tensor
+    bias: Optional[torch.Tensor]
+    mult: float
+
+
+def gated_residual_norm(residual: torch.Tensor, pending: Optional[PendingGated], weight: Optional[torch.Tensor], eps: float, out: torch.Tensor, *,
+                        rows: Optional[torch.Tensor] = None, origin: Optional[torch.Tensor] = None) -> None:
+    """``residual += mult * sigmoid(gate + bias) * values`` (when given), then ``out = rmsnorm(residual) * weight`` (``weight=None``:
+    the residual itself in out's dtype), in one kernel.  ``origin`` (fp32, the residual's shape): its rows go behind, into
+    ``out[:, H:]``.  With ``rows`` only the listed rows are produced and the residual is not written."""
+    what = "gated_residual_norm"
+    T, H = residual.shape
+    R = rows.numel() if rows is not None else T
+    values = gate = bias = mix = at = extra = None
+    K, mult = 1, 0.0
+    if pending is not None:
+        values, gate, bias, mult = pending.values, pending.gate, pending.bias, pending.mult
+        if isinstance(values, WeightedRows):
+            mix, at, extra = values.weights, values.at, values.extra
+            values, K = values.rows, mix.shape[1]
+            if mix.dtype != torch.float32 or not mix.is_contiguous() or mix.shape[0] != T or (at is not None and at.numel() != mix.numel()):
+                raise KernelError(f"{what}: the weights of weighted rows must be contiguous fp32 [tokens, K], with an index entry a row")
+    _need_cuda(what, residual, values, gate, bias, mix, at, extra, weight, out, rows, origin)
+    _need_i32(what, rows, at)
+    if residual.dtype != torch.float32 or not residual.is_contiguous():
+        raise KernelError(f"{what}: the residual must be contiguous fp32")
+    if values is not None and (values.shape != (T * K, H) or not values.is_contiguous() or gate.shape != (T, H) or gate.stride(1) != 1 or gate.dtype != out.dtype):
+        raise KernelError(f"{what}: the values and their gate must have the residual's shape, the gate the activation dtype")
+    if values is not None and ((bias is not None and (bias.numel() != H or not bias.is_contiguous()))
+                               or (extra is not None and (extra.shape != (T, H) or extra.dtype != out.dtype or not extra.is_contiguous()))):
+        raise KernelError(f"{what}: the gate's bias or the extra rows do not fit")
+    wide = 2 * H if origin is not None else H
+    if out.shape[1] != wide or out.shape[0] < R or out.stride(1) != 1 or (weight is not None and (weight.numel() != H or not weight.is_contiguous())):
+        raise KernelError(f"{what}: the output or the norm's weight does not fit")
+    if origin is not None and (origin.dtype != torch.float32 or origin.shape != residual.shape or not origin.is_contiguous()):
+        raise KernelError(f"{what}: the origin must be contiguous fp32 of the residual's shape")
+    fn = _fn("gated_residual", "kb_gated_residual_norm",
+             [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_int, c_float,
+              c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p])
+    _check(fn(residual.data_ptr(), _ptr(values), _is_bf16(values, what) if values is not None else 0, _ptr(mix), _ptr(at), K, _ptr(extra), _ptr(gate),
+              gate.stride(0) if gate is not None else 0, _ptr(bias), _is_bf16(bias, what) if bias is not None else 0, float(mult), _ptr(weight),
+              _is_bf16(weight, what) if weight is not None else 0, float(eps), _ptr(origin), out.data_ptr(), out.stride(0), _is_bf16(out, what),
+              _ptr(rows), R, H, _stream()), what)
 
 
 @dataclass
@@ -1930,11 +2065,11 @@ def moe_route(logits: torch.Tensor, bias: Optional[torch.Tensor], top: int, ids:
 
 
 def moe_route_scores(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, ids: torch.Tensor, weights: torch.Tensor, *,
-                     groups: int = 1, keep: int = 1, scale: float = 1.0, score: str = "softmax") -> None:
+                     groups: int = 1, keep: int = 1, scale: float = 1.0, score: str = "softmax", renormalise: bool = False) -> None:
     """Routing by scores (fp32): s = softmax(logits) over all outputs (``score="sigmoid"``: s = sigmoid(logit), each output by
     itself); the choice runs on s + correction within the ``keep`` best of ``groups`` equal groups of neighbours (a group's
     value: its largest s + correction); the ``top`` best are chosen (ties: the lower index) and weigh s * scale, not
-    renormalised.  ``logits`` may be the leading columns of wider rows (a view ``[:, :n]``)."""
+    renormalised (``renormalise``: divided by the chosen s's sum + 1e-20).  ``logits`` may be the leading columns of wider rows (a view ``[:, :n]``)."""
     _need_cuda("moe_route_scores", logits, correction, ids, weights)
     T, n = logits.shape
     if score not in ("softmax", "sigmoid"):
@@ -1945,9 +2080,9 @@ def moe_route_scores(logits: torch.Tensor, correction: Optional[torch.Tensor], t
         raise KernelError("moe_route_scores: ids and weights must be contiguous [tokens, top]")
     if correction is not None and (correction.numel() != n or not correction.is_contiguous()):
         raise KernelError("moe_route_scores: the correction must have one entry a router output")
-    fn = _fn("moe", "kb_moe_route_scores", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p])
+    fn = _fn("moe", "kb_moe_route_scores", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p])
     _check(fn(logits.data_ptr(), _ptr(correction), _is_bf16(correction, "moe_route_scores") if correction is not None else 0, n, int(top),
-              int(groups), int(keep), float(scale), 1 if score == "sigmoid" else 0, logits.stride(0) if T > 1 else n, ids.data_ptr(),
+              int(groups), int(keep), float(scale), 1 if score == "sigmoid" else 0, 1 if renormalise else 0, logits.stride(0) if T > 1 else n, ids.data_ptr(),
               weights.data_ptr(), T, _stream()), "moe_route_scores")
 
 
@@ -2023,23 +2158,35 @@ def moe_activation(gate_up: torch.Tensor, out: torch.Tensor, *, limit: float, al
     _check(fn(gate_up.data_ptr(), out.data_ptr(), _is_bf16(out, "moe_activation"), rows, wide // 2, float(limit), float(alpha), float(shift), _stream()), "moe_activation")
 
 
-def moe_grouped(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, plan: dict, *, top: int, gated: bool, limit: float = 0.0,
+def _moe_form(what: str, gated: bool, activation: Optional[str]) -> int:
+    """The kernels' code for an expert's product: 0 the second one, 1 the first with the gated unit, 2 the first without gate
+    rows and with relu(up)^2."""
+    if activation is None:
+        return 1 if gated else 0
+    if gated or activation != "relu2":
+        raise KernelError(f"{what}: an ungated expert's activation is relu2, not {activation!r}")
+    return 2
+
+
+def moe_grouped(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, plan: dict, *, top: int, gated: bool, activation: Optional[str] = None, limit: float = 0.0,
                 alpha: float = 1.702, shift: float = 1.0) -> None:
     """The experts' products over a planned step.  ``gated``: ``a`` [tokens, K] activations, ``weight``
     [experts, 2 * N, K] (gate rows, then up rows), ``out`` [pairs, N] in the activations' dtype, rows
-    in the plan's sorted order, after the experts' activation.  Otherwise ``a`` is such an ``out``,
+    in the plan's sorted order, after the experts' activation.  ``activation="relu2"`` (without ``gated``): the same with
+    ``weight`` [experts, N, K], up rows alone, and relu(up)^2.  Otherwise ``a`` is such an ``out``,
     ``weight`` [experts, N, K] and ``out`` fp32 [pairs, N] with row t * top + k for token t's k-th expert."""
     _need_cuda("moe_grouped", a, weight, out)
     experts, rows, K = weight.shape
     N = rows // 2 if gated else rows
+    form = _moe_form("moe_grouped", gated, activation)
     pairs = plan["sorted"].numel()
     if a.dtype != weight.dtype or a.shape[1] != K or a.stride(1) != 1 or not weight.is_contiguous() or not out.is_contiguous():
         raise KernelError("moe_grouped: operands must share a dtype and K, the weight and the output be contiguous")
-    if out.shape != (pairs, N) or out.dtype != (a.dtype if gated else torch.float32):
+    if out.shape != (pairs, N) or out.dtype != (a.dtype if form else torch.float32):
         raise KernelError("moe_grouped: the output does not fit")
     fn = _fn("moe", "kb_moe_grouped", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
                                         c_void_p, c_int, c_float, c_float, c_float, c_int, c_void_p, c_void_p])
-    _check(fn(a.data_ptr(), a.stride(0), plan["sorted"].data_ptr(), int(top), weight.data_ptr(), N, K, _is_bf16(a, "moe_grouped"), 1 if gated else 0,
+    _check(fn(a.data_ptr(), a.stride(0), plan["sorted"].data_ptr(), int(top), weight.data_ptr(), N, K, _is_bf16(a, "moe_grouped"), form,
               plan["tile_expert"].data_ptr(), plan["tile_first"].data_ptr(), plan["tile_pairs"].data_ptr(), plan["num_tiles"].data_ptr(),
               plan["max_tiles"], float(limit), float(alpha), float(shift), experts, out.data_ptr(), _stream()), "moe_grouped")
 
@@ -2060,21 +2207,22 @@ def moe_skinny_ok(tokens: int, hidden: int, intermediate: int, dtype: torch.dtyp
             and max(hidden, intermediate) <= MOE_SKINNY_MAX_WIDTH)
 
 
-def moe_skinny(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, plan: dict, *, top: int, gated: bool, limit: float = 0.0,
+def moe_skinny(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, plan: dict, *, top: int, gated: bool, activation: Optional[str] = None, limit: float = 0.0,
                alpha: float = 1.702, shift: float = 1.0) -> None:
     """``moe_grouped`` for few pairs an expert (bfloat16): the weight rows are the tensor cores' M side, up to 8
     pairs at a time the N side, and the weights are read straight from global memory.  Same operands and results."""
     _need_cuda("moe_skinny", a, weight, out)
     experts, rows, K = weight.shape
     N = rows // 2 if gated else rows
+    form = _moe_form("moe_skinny", gated, activation)
     pairs = plan["sorted"].numel()
     if a.dtype != torch.bfloat16 or weight.dtype != torch.bfloat16 or a.shape[1] != K or a.stride(1) != 1 or not weight.is_contiguous() or not out.is_contiguous():
         raise KernelError("moe_skinny: bfloat16 operands of one K, the weight and the output contiguous")
-    if out.shape != (pairs, N) or out.dtype != (torch.bfloat16 if gated else torch.float32):
+    if out.shape != (pairs, N) or out.dtype != (torch.bfloat16 if form else torch.float32):
         raise KernelError("moe_skinny: the output does not fit")
     fn = _fn("moe", "kb_moe_skinny", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
                                        c_void_p, c_int, c_float, c_float, c_float, c_int, c_void_p, c_void_p])
-    _check(fn(a.data_ptr(), a.stride(0), plan["sorted"].data_ptr(), int(top), weight.data_ptr(), N, K, 1 if gated else 0,
+    _check(fn(a.data_ptr(), a.stride(0), plan["sorted"].data_ptr(), int(top), weight.data_ptr(), N, K, form,
               plan["tile_expert"].data_ptr(), plan["tile_first"].data_ptr(), plan["tile_pairs"].data_ptr(), plan["num_tiles"].data_ptr(),
               plan["max_tiles"], float(limit), float(alpha), float(shift), experts, out.data_ptr(), _stream()), "moe_skinny")
 

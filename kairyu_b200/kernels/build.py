@@ -37,6 +37,8 @@ LIBRARIES: dict[str, list[str]] = {
     "attention_decode_static": [],
     "attention_decode_tma": [],
     "attention_prefill_tc5": [],
+    "talking_attention": [],
+    "gated_residual": [],
     "gemm_f32": [],
     "gemm_skinny": [],
     "gemm_tc5": [],

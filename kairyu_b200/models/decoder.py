@@ -13,6 +13,7 @@ from kairyu_b200.parts.base import (
     HEADS,
     NORMS,
     POSITION_ENCODINGS,
+    STREAM_MAPS,
     CacheView,
     ModelSpec,
     PartSpec,
@@ -39,6 +40,7 @@ class DecoderModel:
         self.embedding_position = (
             POSITION_ENCODINGS.build(spec.embedding_position, **context) if spec.embedding_position is not None else None
         )
+        self.stream_map = STREAM_MAPS.build(spec.stream_map, **context) if spec.stream_map is not None else None
         self.blocks = [
             BLOCKS.build(PartSpec(layer.block), layer=layer, **context) for layer in spec.layers
         ]
@@ -49,6 +51,8 @@ class DecoderModel:
 
     def _validate_schedule(self) -> None:
         written: set[int] = set()
+        if self.stream_map is None and any(call.remaps_stream for call in self.schedule):
+            raise ValueError("a call asks for the stream map, and the model has none")
         for call in self.schedule:
             if not 0 <= call.layer < len(self.blocks):
                 raise ValueError(f"schedule names layer {call.layer}, the model has {len(self.blocks)}")
@@ -73,7 +77,7 @@ class DecoderModel:
         return all(safe(part) for part in self.parts())
 
     def parts(self) -> list[Any]:
-        extra = [self.embedding_position] if self.embedding_position is not None else []
+        extra = [part for part in (self.embedding_position, self.stream_map) if part is not None]
         return [self.embedding, *extra, *self.blocks, self.final_norm, self.head]
 
     def tensor_specs(self) -> list[TensorSpec]:
@@ -87,6 +91,8 @@ class DecoderModel:
         """Weight bytes a decode step reads: every call's block, the final norm
         and the head (embedding rows are gathered, not streamed)."""
         total = sum(self.blocks[call.layer].bytes_streamed() for call in self.schedule)
+        if self.stream_map is not None:
+            total += self.stream_map.bytes_streamed() * sum(1 for call in self.schedule if call.remaps_stream)
         return total + self.final_norm.bytes_streamed() + self.head.bytes_streamed()
 
     # -- cache needs: slot -> specs of the mixer that writes it
@@ -114,9 +120,13 @@ class DecoderModel:
         for index, call in enumerate(calls):
             view = cache_views[(call.cache_slot, call.writes_cache)]
             block = self.blocks[call.layer]
+            if call.remaps_stream:
+                residual, delta = self.stream_map.apply(residual, delta, self.embedding.origin(ctx), ctx), None
             if getattr(block, "takes_next_norm", False):
                 # a block may begin the first norm of the block that runs next, if that block offers one
-                following = self.blocks[calls[index + 1].layer] if index + 1 < len(calls) else None
+                # (not across a stream map: the norm reads what the map gives)
+                after = calls[index + 1] if index + 1 < len(calls) else None
+                following = self.blocks[after.layer] if after is not None and not after.remaps_stream else None
                 offer = getattr(following, "prenorm_target", None)
                 residual, delta = block.forward(residual, delta, ctx, view, next_norm=offer(ctx) if offer else None)
             else:

@@ -2,7 +2,8 @@
 built-in parts; more can be registered from outside with the same decorators."""
 
 from kairyu_b200.parts import (  # noqa: F401  (registration)
-    attention, block, delta_rule, diff_attention, embedding, ffn, gated_attention, latent_attention, learned_positions, moe, norm, rope, side_by_side, state_space,
+    attention, block, delta_rule, diff_attention, embedding, ffn, gated_attention, latent_attention, learned_positions, moe, norm, rope, side_by_side, state_space, stream_map,
+    talking_attention,
 )
 from kairyu_b200.parts.base import (
     BLOCKS,
@@ -12,6 +13,7 @@ from kairyu_b200.parts.base import (
     MIXERS,
     NORMS,
     POSITION_ENCODINGS,
+    STREAM_MAPS,
     Block,
     CacheView,
     FeedForward,
@@ -26,11 +28,12 @@ from kairyu_b200.parts.base import (
     PositionEncoding,
     StateSpec,
     StepContext,
+    StreamMap,
     TensorSpec,
 )
 
 __all__ = [
-    "BLOCKS", "EMBEDDINGS", "FEED_FORWARDS", "HEADS", "MIXERS", "NORMS", "POSITION_ENCODINGS",
+    "BLOCKS", "EMBEDDINGS", "FEED_FORWARDS", "HEADS", "MIXERS", "NORMS", "POSITION_ENCODINGS", "STREAM_MAPS",
     "Block", "CacheView", "FeedForward", "LayerCall", "LayerSpec", "Mixer", "ModelSpec", "Norm",
-    "PagedKVSpec", "Part", "PartSpec", "PositionEncoding", "StateSpec", "StepContext", "TensorSpec",
+    "PagedKVSpec", "Part", "PartSpec", "PositionEncoding", "StateSpec", "StepContext", "StreamMap", "TensorSpec",
 ]

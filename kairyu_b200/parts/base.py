@@ -59,6 +59,8 @@ class LayerSpec:
     # norms on the sub-layers' OUTPUTS, for arrangements that norm on both sides of a sub-layer
     mixer_post_norm: Optional[PartSpec] = None
     ffn_post_norm: Optional[PartSpec] = None
+    # what else an arrangement wants to know (tensor names and constants of its own)
+    options: Mapping[str, Any] = field(default_factory=dict, hash=False)
 
 
 @dataclass(frozen=True)
@@ -68,12 +70,14 @@ class LayerCall:
     ``layer`` indexes ``ModelSpec.layers`` (a layer may be named by several
     calls).  ``cache_slot`` is the cache this call's mixer uses; a call with
     ``writes_cache=False`` reads a slot that an earlier call of the same step
-    wrote (one layer reading another layer's keys and values).
+    wrote (one layer reading another layer's keys and values).  ``remaps_stream``:
+    the model's stream map (``ModelSpec.stream_map``) runs right before the layer.
     """
 
     layer: int
     cache_slot: int
     writes_cache: bool = True
+    remaps_stream: bool = False
 
 
 @dataclass(frozen=True)
@@ -89,6 +93,9 @@ class ModelSpec:
     # A position encoding that acts on the embedding (learned absolute positions and the like);
     # rotary kinds belong to the mixers that use them.
     embedding_position: Optional[PartSpec] = None
+    # A map of the whole residual stream that runs before the calls that ask for it
+    # (``LayerCall.remaps_stream``); it also sees the embedding output, which the embedding then keeps.
+    stream_map: Optional[PartSpec] = None
 
 
 # --------------------------------------------------------------------------- weights
@@ -121,13 +128,15 @@ class PagedKVSpec:
     keeps the last ``window`` positions (older pages go back to the pool).
     ``v_head_dim``: the width of a value row where it differs from a key row's
     (a mixer whose values are narrower than its keys; None: the same; 0: no value
-    rows at all, for a mixer whose keys and values are products of one cached row).  Slots
-    whose specs are equal share a group: pages of one geometry, one block table."""
+    rows at all, for a mixer whose keys and values are products of one cached row).
+    ``keep_first``: with a window, the sequence's first tokens that every later query still sees;
+    their pages stay as long as the request lives.  Slots whose specs are equal share a group: pages of one geometry, one block table."""
 
     num_kv_heads: int
     head_dim: int
     window: int | None = None
     v_head_dim: int | None = None
+    keep_first: int = 0
 
     @property
     def value_dim(self) -> int:
@@ -231,6 +240,15 @@ class Norm(Part):
         raise NotImplementedError
 
 
+class StreamMap(Part):
+    """A map of the residual stream itself, between two layers."""
+
+    def apply(self, residual: torch.Tensor, delta: Any, origin: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        """The new stream (fp32) from the old one, what is still to be added to it (``delta``), and the
+        embedding output ``origin`` (fp32)."""
+        raise NotImplementedError
+
+
 class PositionEncoding(Part):
     def rotary_tables(self) -> tuple[torch.Tensor, torch.Tensor] | None:
         """(cos, sin), each [max_positions, rotary_dim/2] fp32, or None."""
@@ -314,3 +332,4 @@ POSITION_ENCODINGS = Registry("position encoding")
 BLOCKS = Registry("block arrangement")
 EMBEDDINGS = Registry("embedding")
 HEADS = Registry("output head")
+STREAM_MAPS = Registry("stream map")

@@ -188,6 +188,79 @@ class ParallelBlock(Block):
         return residual, kernels.PendingSums(mixed, self.ffn.forward(normed, ctx))
 
 
+@BLOCKS.register("gated_residual")
+class GatedResidualBlock(Block):
+    """``h = norm1(x); x += m * sigmoid(R1 h + b1) * mixer(h);  h = norm2(x); x += m * sigmoid(R2 h + b2) * ffn(h)``: each
+    sub-layer's result is gated element by element by a product of what the sub-layer reads, and scaled by one constant
+    (``LayerSpec.options``: ``gate_names``, the two gates' tensors, each with a bias ``.b``, and ``residual_mult``).  A layer
+    may have no feed-forward.
+
+    The residual is fp32.  A sub-layer's output, its gate's rows and its bias travel on (``kernels.PendingGated``), and the kernel
+    of the norm that reads the stream next forms the gate, adds and norms, so a gated sum costs no kernel of its own; a mixture
+    hands over its experts' rows before their sum and that kernel adds them too.  A mixer that takes further rows into its own
+    input product (``carry_rows``) computes the gate there; elsewhere it is a product of its own."""
+
+    graph_safe = True
+
+    def __init__(self, *, layer: LayerSpec, dtype: torch.dtype, device: str, shared: dict, **_: object) -> None:
+        context = dict(dtype=dtype, device=device, shared=shared)
+        self.dtype = dtype
+        self.gate_names = tuple(layer.options["gate_names"])
+        self.mult = float(layer.options.get("residual_mult", 1.0))
+        self.size = int(layer.mixer_norm.params["size"])
+        self.mixer_norm = NORMS.build(layer.mixer_norm, **context)
+        self.mixer = MIXERS.build(layer.mixer, **context)
+        self.ffn_norm = NORMS.build(layer.ffn_norm, **context) if layer.ffn is not None else None
+        self.ffn = FEED_FORWARDS.build(layer.ffn, **context) if layer.ffn is not None else None
+        self._parts = tuple(part for part in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if part is not None)
+        self._carried = hasattr(self.mixer, "carry_rows")
+        self._gates: list[Optional[torch.Tensor]] = [None, None]  # weights of gates that are products of their own
+        self._biases: list[Optional[torch.Tensor]] = [None, None]
+
+    def _sub_layers(self) -> int:
+        return 1 if self.ffn is None else 2
+
+    def tensor_specs(self) -> list[TensorSpec]:
+        specs = [spec for part in self._parts for spec in part.tensor_specs()]
+        for name in self.gate_names[: self._sub_layers()]:
+            specs += [TensorSpec(name, (self.size, self.size)), TensorSpec(f"{name}.b", (self.size,), role="vector", init="normal")]
+        return specs
+
+    def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        for index, name in enumerate(self.gate_names[: self._sub_layers()]):
+            self._gates[index] = tensors[name].contiguous()
+            self._biases[index] = tensors[f"{name}.b"].contiguous()
+        if self._carried:
+            self.mixer.carry_rows(self._gates[0])
+            self._gates[0] = None
+        for part in self._parts:
+            part.load(tensors)
+
+    def bytes_streamed(self) -> int:
+        own = sum(t.numel() * t.element_size() for t in (*self._gates, *self._biases) if t is not None)
+        return own + sum(part.bytes_streamed() for part in self._parts)
+
+    def _gate(self, index: int, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        rows = ctx.workspace.buffer(f"block.gate{index}", h.shape[0], self.size, self.dtype)
+        kernels.linear(h, self._gates[index], None, rows)
+        return rows
+
+    def forward(self, residual: torch.Tensor, delta, ctx: StepContext, cache: CacheView):
+        normed = self.mixer_norm.apply(residual, delta, ctx)
+        gate = None if self._carried else self._gate(0, normed, ctx)
+        mixed = self.mixer.forward(normed, ctx, cache)
+        pending = kernels.PendingGated(mixed, self.mixer.carried_rows(ctx) if self._carried else gate, self._biases[0], self.mult)
+        if self.ffn is None:
+            return residual, pending
+        normed = self.ffn_norm.apply(residual, pending, ctx)
+        gate = self._gate(1, normed, ctx)
+        if getattr(self.ffn, "weighted_rows_and_extra", False):
+            output = self.ffn.forward(normed, ctx, combine=False)
+        else:
+            output = self.ffn.forward(normed, ctx)
+        return residual, kernels.PendingGated(output, gate, self._biases[1], self.mult)
+
+
 @BLOCKS.register("sandwich_norm")
 class SandwichNormBlock(Block):
     """``x += post1(mixer(pre1(x))); x += post2(ffn(pre2(x)))``: a norm before and a norm after each sub-layer.  A layer

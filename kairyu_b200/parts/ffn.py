@@ -80,7 +80,8 @@ class SwiGLU(FeedForward):
 class UngatedMLP(FeedForward):
     """``down(act(up(x)))`` without a gate and without biases.  ``activation``: ``relu2`` (the square of
     relu), ``gelu_tanh`` or ``silu``; it runs in 32-bit on the up product's rows, with one rounding at
-    the store.  ``up_name`` / ``down_name``: the two tensors' names under ``prefix``."""
+    the store.  ``up_name`` / ``down_name``: the two tensors' names under ``prefix``; ``tag`` names the workspace
+    buffers (two that are alive at once take different tags)."""
 
     graph_safe = True
 
@@ -93,6 +94,7 @@ class UngatedMLP(FeedForward):
         activation: str,
         up_name: str = "up",
         down_name: str = "down",
+        tag: str = "mlp",
         dtype: torch.dtype,
         device: str,
         **_: object,
@@ -105,6 +107,7 @@ class UngatedMLP(FeedForward):
         self.activation = activation
         self.up_name = f"{prefix}.{up_name}"
         self.down_name = f"{prefix}.{down_name}"
+        self.tag = tag
         self.dtype = dtype
         self.w_up: Optional[torch.Tensor] = None
         self.w_down: Optional[torch.Tensor] = None
@@ -131,13 +134,13 @@ class UngatedMLP(FeedForward):
         adds its result to the residual and returns the ``PreNormed`` for the next norm."""
         tokens = x.shape[0]
         ws = ctx.workspace
-        hidden = ws.buffer("mlp.hidden", tokens, self.intermediate_size, self.dtype)
+        hidden = ws.buffer(f"{self.tag}.hidden", tokens, self.intermediate_size, self.dtype)
         kernels.linear(x, self.w_up, None, hidden)
         kernels.activation(hidden, hidden, self.activation)
         if fold is not None:
             kernels.linear(hidden, self.w_down, None, None, fold=fold)
             return fold.result()
-        out = ws.buffer("mlp.out", tokens, self.hidden_size, self.dtype)
+        out = ws.buffer(f"{self.tag}.out", tokens, self.hidden_size, self.dtype)
         kernels.linear(hidden, self.w_down, None, out)
         return out
 

@@ -6,7 +6,8 @@ index); the weights are the softmax over the chosen logits only.  ``routing="sco
 outputs; the choice runs on s + a stored ``correction`` within the ``groups_keep`` best of ``groups`` equal groups of
 neighbouring outputs (a group's value is its largest s + correction); the weights are s * ``route_scale``, not
 renormalised.  ``score_function="sigmoid"`` takes s = sigmoid(logit), each output by itself, in place of the softmax;
-``correction=False`` means the file stores none.  The last ``num_identity`` router outputs are identity experts: no
+``correction=False`` means the file stores none; ``renormalise=True`` divides a token's weights by the sum of its chosen scores
+(+ 1e-20) before ``route_scale``.  The last ``num_identity`` router outputs are identity experts: no
 tensors, their output is the token's row itself (``num_experts`` counts the experts with weights).
 
 ``weight_on="input"``: the router's weight multiplies the expert's input, ``sum_k expert_k(w_k x)``, instead of its output
@@ -14,12 +15,13 @@ tensors, their output is the token's row itself (``num_experts`` counts the expe
 added up unweighted.
 
 ``shared_expert`` (a dict: ``intermediate_size``, optional ``limit`` / ``alpha`` / ``shift``, ``gate``): one more expert of the same
-form that every token runs (tensors ``<prefix>.shared.gate`` / ``.up`` / ``.down``); with ``gate`` its output is multiplied
+form that every token runs (tensors ``<prefix>.shared.gate`` / ``.up`` / ``.down``, without ``.gate`` for ungated experts); with ``gate`` its output is multiplied
 by ``sigmoid(w_sg . x)``, one number a token (tensor ``<prefix>.shared.sg``, [1, hidden]), which is computed with the router's
 logits, in 32-bit, as one more row of that product.
 
 An expert is ``W_down(a * sigmoid(alpha a) * (b + shift))`` with ``a = min(W_gate x, limit)`` and
 ``b = clamp(W_up x, -limit, limit)``; ``limit=None``, ``alpha=1``, ``shift=0`` give ``silu(W_gate x) * (W_up x)``.
+``activation="relu2"``: experts without a gate, ``W_down relu(W_up x)^2`` (tensors ``.up`` and ``.down`` alone).
 
 A step's (token, expert) pairs are sorted by expert on the device (``csrc/moe.cu``).  In bfloat16
 with rows of whole 16 bytes a step of up to 16 tokens runs the weight-streaming kernel for few pairs
@@ -30,7 +32,8 @@ and the rows left in sorted order; float32 and other sizes run this package's ow
 (gate and up with the activation in the epilogue, then down).  Nothing comes back to the host, so
 the work can sit in a captured graph.  Either way there is one row per pair at the end;
 ``forward(..., combine=False)`` hands those, the router's weights and where each row lies on
-(``kernels.WeightedRows``) for a kernel that adds them on its way, otherwise they are added here.
+(``kernels.WeightedRows``) for a kernel that adds them on its way (with an ungated-by-a-number shared expert's rows beside
+them), otherwise they are added here.
 """
 
 from __future__ import annotations
@@ -56,7 +59,7 @@ class MixtureOfExperts(FeedForward):
         intermediate_size: int,
         num_experts: int,
         top: int,
-        limit: Optional[float],
+        limit: Optional[float] = None,
         alpha: float = 1.702,
         shift: float = 1.0,
         router_bias: bool = True,
@@ -69,6 +72,8 @@ class MixtureOfExperts(FeedForward):
         correction: bool = True,
         weight_on: str = "output",
         shared_expert: Optional[Mapping[str, object]] = None,
+        renormalise: bool = False,
+        activation: Optional[str] = None,
         dtype: torch.dtype,
         device: str,
         **_: object,
@@ -92,6 +97,12 @@ class MixtureOfExperts(FeedForward):
             raise ValueError("a gated shared expert comes with routing by scores")
         if weight_on == "input" and num_identity:
             raise ValueError("identity experts take the router's weight on their output")
+        if activation not in (None, "relu2"):
+            raise ValueError(f"an ungated expert's activation is relu2, not {activation!r}")
+        if renormalise and routing != "scores":
+            raise ValueError("weights divided by their sum come with routing by scores (a softmax over the chosen logits sums to one)")
+        self.activation = activation
+        self.renormalise = bool(renormalise)
         self.score_function = score_function
         self.has_correction = correction and routing == "scores"
         self.weight_on_input = weight_on == "input"
@@ -100,9 +111,10 @@ class MixtureOfExperts(FeedForward):
         if shared_expert is not None:
             options = dict(shared_expert)
             self.shared_gate = bool(options.pop("gate", False))
-            self.shared = FEED_FORWARDS.build(
-                PartSpec("gated_unit", prefix=f"{prefix}.shared", hidden_size=hidden_size, tag="moe.shared", **options), dtype=dtype, device=device
-            )
+            form = PartSpec("gated_unit", prefix=f"{prefix}.shared", hidden_size=hidden_size, tag="moe.shared", **options)
+            if activation is not None:
+                form = PartSpec("mlp", prefix=f"{prefix}.shared", hidden_size=hidden_size, tag="moe.shared", activation=activation, **options)
+            self.shared = FEED_FORWARDS.build(form, dtype=dtype, device=device)
         self.w_shared_gate: Optional[torch.Tensor] = None
         self.routing = routing
         self.num_identity = num_identity
@@ -113,6 +125,8 @@ class MixtureOfExperts(FeedForward):
         self.shift = float(shift)
         # a kernel that adds the rows itself (kernels.WeightedRows) knows nothing of identity experts
         self.weighted_rows = num_identity == 0 and not self.weight_on_input and self.shared is None
+        # ... and one that also adds an always-on expert's rows takes those beside them
+        self.weighted_rows_and_extra = num_identity == 0 and not self.weight_on_input and not self.shared_gate
         self.prefix = prefix
         self.hidden_size = hidden_size
         self.intermediate_size = intermediate_size
@@ -125,18 +139,17 @@ class MixtureOfExperts(FeedForward):
         self.correction: Optional[torch.Tensor] = None
         self.w_router: Optional[torch.Tensor] = None
         self.b_router: Optional[torch.Tensor] = None
-        self.w_gate_up: Optional[torch.Tensor] = None  # [experts, 2 * intermediate, hidden]: gate rows, then up rows
+        # [experts, 2 * intermediate, hidden]: gate rows, then up rows; ungated experts: [experts, intermediate, hidden]
+        self.w_gate_up: Optional[torch.Tensor] = None
         self.w_down: Optional[torch.Tensor] = None     # [experts, hidden, intermediate]
 
     def tensor_specs(self) -> list[TensorSpec]:
         p, h, f = self.prefix, self.hidden_size, self.intermediate_size
         specs = []
         for e in range(self.num_experts):
-            specs += [
-                TensorSpec(f"{p}.e{e}.gate", (f, h)),
-                TensorSpec(f"{p}.e{e}.up", (f, h)),
-                TensorSpec(f"{p}.e{e}.down", (h, f)),
-            ]
+            if self.activation is None:
+                specs.append(TensorSpec(f"{p}.e{e}.gate", (f, h)))
+            specs += [TensorSpec(f"{p}.e{e}.up", (f, h)), TensorSpec(f"{p}.e{e}.down", (h, f))]
         specs.append(TensorSpec(f"{p}.router", (self.num_outputs, h)))
         if self.has_correction:
             specs.append(TensorSpec(f"{p}.correction", (self.num_outputs,), role="vector", init="normal"))
@@ -151,9 +164,8 @@ class MixtureOfExperts(FeedForward):
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         p = self.prefix
         experts = range(self.num_experts)
-        self.w_gate_up = torch.stack(
-            [torch.cat([tensors[f"{p}.e{e}.gate"], tensors[f"{p}.e{e}.up"]], dim=0) for e in experts], dim=0
-        ).contiguous()
+        first = ("up",) if self.activation is not None else ("gate", "up")
+        self.w_gate_up = torch.stack([torch.cat([tensors[f"{p}.e{e}.{name}"] for name in first], dim=0) for e in experts], dim=0).contiguous()
         self.w_down = torch.stack([tensors[f"{p}.e{e}.down"] for e in experts], dim=0).contiguous()
         self.w_router = tensors[f"{p}.router"].contiguous()
         if self.shared is not None:
@@ -181,12 +193,14 @@ class MixtureOfExperts(FeedForward):
         weights = ws.buffer("moe.weights", tokens, top, torch.float32)
         if self.routing == "scores":
             kernels.moe_route_scores(logits[:, :experts], self.correction, top, ids, weights, groups=self.groups, keep=self.groups_keep,
-                                     scale=self.route_scale, score=self.score_function)
+                                     scale=self.route_scale, score=self.score_function, renormalise=self.renormalise)
         else:
             kernels.moe_route(logits, self.b_router, top, ids, weights)
         pairs = tokens * top
         plan = kernels.moe_plan(ids, experts, ws.flat("moe.plan", kernels.moe_plan_size(pairs, experts), torch.int32))
-        unit = dict(limit=self.limit, alpha=self.alpha, shift=self.shift)
+        unit = dict(gated=True, limit=self.limit, alpha=self.alpha, shift=self.shift)
+        if self.activation is not None:
+            unit = dict(gated=False, activation=self.activation)
         library = not kernels.moe_skinny_ok(tokens, self.hidden_size, self.intermediate_size, self.dtype) \
             and kernels.moe_library_products_ok(self.hidden_size, self.intermediate_size, self.dtype)
         if self.weight_on_input and not library:
@@ -198,7 +212,7 @@ class MixtureOfExperts(FeedForward):
             # a decode-sized step: an expert has a handful of pairs and its weights stream once (gate and up with the
             # activation in the epilogue, then down)
             hidden = ws.buffer("moe.hidden", pairs, self.intermediate_size, self.dtype)
-            kernels.moe_skinny(x, self.w_gate_up, hidden, plan, top=top, gated=True, **unit)
+            kernels.moe_skinny(x, self.w_gate_up, hidden, plan, top=top, **unit)
             rows, at = ws.buffer("moe.rows", pairs, self.hidden_size, torch.float32), None
             kernels.moe_skinny(hidden, self.w_down, rows, plan, top=top, gated=False)
         elif kernels.moe_library_products_ok(self.hidden_size, self.intermediate_size, self.dtype):
@@ -212,17 +226,20 @@ class MixtureOfExperts(FeedForward):
                 kernels.gather_rows(x, plan["token_of"], gathered)
             gate_up = kernels.moe_library_product(gathered, self.w_gate_up, ends)
             hidden = ws.buffer("moe.hidden", pairs, self.intermediate_size, self.dtype)
-            kernels.moe_activation(gate_up, hidden, **unit)
+            if self.activation is not None:
+                kernels.activation(gate_up, hidden, self.activation)
+            else:
+                kernels.moe_activation(gate_up, hidden, limit=self.limit, alpha=self.alpha, shift=self.shift)
             rows, at = kernels.moe_library_product(hidden, self.w_down, ends), plan["place_of"]
         else:
             hidden = ws.buffer("moe.hidden", pairs, self.intermediate_size, self.dtype)
-            kernels.moe_grouped(x, self.w_gate_up, hidden, plan, top=top, gated=True, **unit)
+            kernels.moe_grouped(x, self.w_gate_up, hidden, plan, top=top, **unit)
             rows, at = ws.buffer("moe.rows", pairs, self.hidden_size, torch.float32), None
             kernels.moe_grouped(hidden, self.w_down, rows, plan, top=top, gated=False)
         if not combine:
-            if not self.weighted_rows:
-                raise ValueError("a mixture with identity experts, weights on the experts' inputs or a shared expert adds its rows itself")
-            return kernels.WeightedRows(rows, weights, at)
+            if not self.weighted_rows_and_extra:
+                raise ValueError("a mixture with identity experts, weights on the experts' inputs or a gated shared expert adds its rows itself")
+            return kernels.WeightedRows(rows, weights, at, self.shared.forward(tokens_rows, ctx) if self.shared is not None else None)
         out = ws.buffer("moe.out", tokens, self.hidden_size, self.dtype)
         extras = {}
         if self.shared is not None:

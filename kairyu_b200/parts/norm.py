@@ -15,17 +15,19 @@ class RMSNorm(Norm):
     """``y = x * rsqrt(mean(x^2) + eps) * (offset + weight)`` with fp32 statistics.  ``offset`` is 0 unless
     given; a file that stores its norm weights around zero names 1, and the sum is then formed once,
     at loading, in 32-bit, and held so.  ``scalar``: the weight is ONE number for all coordinates (a tensor
-    without dimensions); it is spread over the width once, at loading, in 32-bit."""
+    without dimensions); it is spread over the width once, at loading, in 32-bit.  ``gain``: a factor on the norm's
+    whole result (a model that scales its logits puts it on its last norm); it is multiplied into the weight the same way."""
 
     graph_safe = True
 
     def __init__(self, *, name: str, size: int, eps: float, dtype: torch.dtype, device: str, offset: float = 0.0, scalar: bool = False,
-                 **_: object) -> None:
+                 gain: float = 1.0, **_: object) -> None:
         self.name = name  # full tensor name of the weight
         self.size = size
         self.eps = float(eps)
         self.offset = float(offset)
         self.scalar = bool(scalar)
+        self.gain = float(gain)
         self.dtype = dtype
         self.device = device
         self.weight: Optional[torch.Tensor] = None
@@ -40,6 +42,8 @@ class RMSNorm(Norm):
             self.weight = self.weight.float().reshape(1).expand(self.size).contiguous()
         if self.offset != 0.0:
             self.weight = (self.weight.float() + self.offset).contiguous()
+        if self.gain != 1.0:
+            self.weight = (self.weight.float() * self.gain).contiguous()
 
     def bytes_streamed(self) -> int:
         return self.weight.numel() * self.weight.element_size()
@@ -57,6 +61,9 @@ class RMSNorm(Norm):
         out = ctx.workspace.buffer("norm.out" if rows is None else "norm.rows.out", count, self.size, self.dtype)
         if isinstance(delta, kernels.PendingNormed):  # a normed sub-layer output still to be added: one kernel for both norms
             kernels.sandwich_norm(residual, delta, self.weight, self.eps, out, rows=rows)
+            return out
+        if isinstance(delta, kernels.PendingGated):  # a gated sub-layer output still to be added
+            kernels.gated_residual_norm(residual, delta, self.weight, self.eps, out, rows=rows)
             return out
         kernels.rmsnorm(residual, self.weight, self.eps, out, delta=delta, rows=rows)
         return out

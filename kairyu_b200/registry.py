@@ -71,6 +71,9 @@ def _register_builtin() -> None:
     from kairyu_b200.models import tapasun
 
     register_architecture("Tapasun", tapasun.parse_tapasun, tapasun.tapasun_spec)
+    from kairyu_b200.models import koravik
+
+    register_architecture("Koravik", koravik.parse_koravik, koravik.koravik_spec)
 
 
 _register_builtin()
