@@ -666,6 +666,83 @@ def talking_prepare(
               _stream()), what)
 
 
+def talking_attention_supported(num_q_heads: int, num_kv_heads: int, head_dim: int) -> bool:
+    """Sizes that the tensor-core kernels of attention over one wide key row take (csrc/talking_attention_tc5.cu: ``supported``,
+    csrc/talking_attention_decode.cu: ``td_shape``): heads of a multiple of 16 up to 128 columns, key rows that fit beside their
+    rings of buffers in shared memory (up to about 640 columns), up to 16 query heads a key/value head and 64 in all."""
+    if num_kv_heads < 1 or num_q_heads % num_kv_heads or num_q_heads // num_kv_heads > 16 or num_q_heads > 64 or head_dim % 16 or not 16 <= head_dim <= 128:
+        return False
+    width = num_kv_heads * head_dim
+    band = 128 * 128
+    bands, value_bands = -(-width // 64), -(-head_dim // 64)
+    if (227 * 1024 - 216 - (bands + value_bands) * band) // band < 2:
+        return False
+    rows, stride = 16 * -(-num_q_heads // 16), width + 8
+    two_stages = (rows * stride + 2 * 64 * stride + rows * 40) * 2 + (2 * rows * 34 + 3 * rows) * 4
+    return width <= 1024 and two_stages <= 220 * 1024
+
+
+def talking_attention_tile(num_q_heads: int, num_kv_heads: int) -> int:
+    """Queries a tile of the kernel for prompt portions: a tile's 128 rows are the query heads of one key/value head."""
+    return 128 // (num_q_heads // num_kv_heads)
+
+
+def talking_attention(
+    queries: torch.Tensor,
+    out: torch.Tensor,
+    k_cache: torch.Tensor,
+    v_cache: torch.Tensor,
+    *,
+    ctx: object,
+    block_table: torch.Tensor,
+    num_q_heads: int,
+    scale: float,
+    window: int = 0,
+    keep_first: int = 0,
+    flag: Optional[torch.Tensor] = None,
+) -> None:
+    """Attention of a step's tokens with the mixed queries of ``talking_prepare`` (bfloat16, tensor cores): head h scores a position by
+    its row of ``queries`` times the position's keys side by side, and takes the values of its own key/value head; a token sees
+    itself, the ``window - 1`` before it (0: all) and the first ``keep_first``.  Prompt portions go tile by tile
+    (``ctx.tiles[talking_attention_tile(...)]``), single-token rows (``ctx.decode_rows``) with their keys split over as many blocks as
+    fill the device.  Caches [pages, page, kv_heads, dim]."""
+    what = "talking_attention"
+    _need_cuda(what, queries, out, k_cache, v_cache, block_table, flag)
+    _need_i32(what, block_table)
+    num_pages, page_size, num_kv_heads, head_dim = k_cache.shape
+    if queries.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or k_cache.dtype != torch.bfloat16 or v_cache.dtype != torch.bfloat16 \
+            or v_cache.shape != k_cache.shape or not (k_cache.is_contiguous() and v_cache.is_contiguous()) or queries.stride(1) != 1 or out.stride(1) != 1:
+        raise KernelError(f"{what}: bfloat16, contiguous caches of one geometry, unit inner strides")
+    if not talking_attention_supported(num_q_heads, num_kv_heads, head_dim):
+        raise KernelError(f"{what}: {num_q_heads} heads over {num_kv_heads} of {head_dim} columns are not supported")
+    if queries.shape[1] != num_q_heads * num_kv_heads * head_dim or out.shape[1] < num_q_heads * head_dim or out.shape[0] != queries.shape[0]:
+        raise KernelError(f"{what}: the queries or the output do not fit the heads")
+    tiles = ctx.tiles[talking_attention_tile(num_q_heads, num_kv_heads)]
+    if tiles[0]:
+        fn = _fn("talking_attention_tc5", "kb_talking_attention_tc5",
+                 [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
+                  c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p])
+        _check(fn(queries.data_ptr(), queries.stride(0), out.data_ptr(), out.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), ctx.qo_indptr.data_ptr(),
+                  ctx.seq_lens.data_ptr(), block_table.data_ptr(), block_table.shape[1], tiles[1].data_ptr(), tiles[2].data_ptr(), int(tiles[0]),
+                  num_q_heads, num_kv_heads, head_dim, page_size, num_pages, float(scale), int(window), int(keep_first), _ptr(flag), _stream()), what)
+    count = ctx.num_decode_rows
+    if count:
+        keys = ctx.max_seq_len if window <= 0 else min(ctx.max_seq_len, window + keep_first)
+        splits_fn = _fn("talking_attention_decode", "kb_talking_decode_splits", [c_int] * 5)
+        splits = int(splits_fn(count, int(keys), num_q_heads, num_kv_heads, head_dim))
+        part_o = part_ml = None
+        if splits > 1:
+            part_o = ctx.workspace.flat("talk.part_o", splits * count * num_q_heads * head_dim, torch.float32)
+            part_ml = ctx.workspace.flat("talk.part_ml", splits * count * num_q_heads * 2, torch.float32)
+        fn = _fn("talking_attention_decode", "kb_talking_decode",
+                 [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                  c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p])
+        _check(fn(queries.data_ptr(), queries.stride(0), out.data_ptr(), out.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), ctx.seq_lens.data_ptr(),
+                  block_table.data_ptr(), block_table.shape[1], ctx.decode_rows.data_ptr(), ctx.decode_tokens.data_ptr(), int(count), num_q_heads,
+                  num_kv_heads, head_dim, page_size, num_pages, float(scale), int(window), int(keep_first), splits, _ptr(part_o), _ptr(part_ml),
+                  _stream()), what, launches=2 if splits > 1 else 1)
+
+
 DIFF_ATTENTION_TILE = 64  # queries a tile of the tensor-core kernel for prompt portions
 
 

@@ -38,6 +38,8 @@ LIBRARIES: dict[str, list[str]] = {
     "attention_decode_tma": [],
     "attention_prefill_tc5": [],
     "talking_attention": [],
+    "talking_attention_tc5": [],
+    "talking_attention_decode": [],
     "gated_residual": [],
     "gemm_f32": [],
     "gemm_skinny": [],

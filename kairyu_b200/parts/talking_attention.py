@@ -12,7 +12,9 @@ One product gives ``q | k | v`` (``values="keys"``: ``q | k``, a value is the ke
 The mix is linear in the queries, so it costs no pass over the scores: ``kernels.talking_prepare`` mixes the turned queries
 in 32-bit (head h gets one row that spans every key/value head's key, ``num_kv_heads * head_dim`` columns) and attention
 is that of heads which share one wide key row a position and take their values from their own key/value head.  Cached per
-token and key/value head: the turned key and the value.
+token and key/value head: the turned key and the value.  bfloat16 of sizes ``kernels.talking_attention_supported`` names runs
+on tensor cores (prompt portions in tiles of queries, single tokens with their keys split over blocks); everything else
+runs the 32-bit-arithmetic kernel.
 
 Tensors under ``prefix``: ``q``, ``k``, ``o``, ``talk`` [heads, heads], and ``v`` with ``values="projection"``.
 ``carry_rows`` takes further weight rows into the input product for the block around the mixer (a gate that reads
@@ -121,6 +123,13 @@ class TalkingAttention(Mixer):
     def cache_specs(self) -> tuple[Any, ...]:
         return (PagedKVSpec(self.num_kv_heads, self.head_dim, self.window, keep_first=self.keep_first),)
 
+    def _tensor_cores(self) -> bool:
+        """bfloat16 and sizes the tensor-core kernels take; float32 and other sizes run the 32-bit-arithmetic kernel."""
+        return self.dtype == torch.bfloat16 and kernels.talking_attention_supported(self.num_heads, self.num_kv_heads, self.head_dim)
+
+    def query_tile_sizes(self) -> tuple[int, ...]:
+        return (kernels.talking_attention_tile(self.num_heads, self.num_kv_heads),) if self._tensor_cores() else ()
+
     # -- compute
     def _packed(self, ctx: StepContext) -> torch.Tensor:
         return ctx.workspace.buffer("talk.packed", ctx.num_tokens, self.packed_width, self.dtype)
@@ -140,12 +149,14 @@ class TalkingAttention(Mixer):
             k_cache=cache.k if cache.writes else None, v_cache=cache.v if cache.writes else None, flag=ctx.error_flag,
         )
         mixed = ws.buffer("talk.mixed", tokens, self.q_size, self.dtype)
-        # a position's keys side by side are one key row that all heads share
-        wide_keys = cache.k.view(cache.k.shape[0], cache.k.shape[1], 1, self.kv_size)
-        kernels.diff_attention_generic(
-            queries, mixed, wide_keys, cache.v, positions=ctx.positions, row_ids=ctx.row_ids, block_table=block_table, num_q_heads=self.num_heads,
-            maps=1, scale=self.scale, window=self.window or 0, keep_first=self.keep_first, flag=ctx.error_flag,
-        )
+        constants = dict(num_q_heads=self.num_heads, scale=self.scale, window=self.window or 0, keep_first=self.keep_first, flag=ctx.error_flag)
+        if self._tensor_cores() and not ctx.extras.get("force_generic_attention", False):
+            kernels.talking_attention(queries, mixed, cache.k, cache.v, ctx=ctx, block_table=block_table, **constants)
+        else:
+            # a position's keys side by side are one key row that all heads share
+            wide_keys = cache.k.view(cache.k.shape[0], cache.k.shape[1], 1, self.kv_size)
+            kernels.diff_attention_generic(queries, mixed, wide_keys, cache.v, positions=ctx.positions, row_ids=ctx.row_ids, block_table=block_table,
+                                           maps=1, **constants)
         out = ws.buffer("talk.out", tokens, self.hidden_size, self.dtype)
         kernels.linear(mixed, self.w_o, None, out)
         return out
