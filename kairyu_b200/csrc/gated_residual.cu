@@ -13,8 +13,9 @@
 // strides and the weights' alignment alone, never on the batch.
 #include "common.cuh"
 
-#define GR_THREADS 256
-#define GR_CHUNKS 4  // four-column groups a thread of the vector form keeps: rows of up to 4 * 4 * 256 columns
+#define GR_THREADS 256      // of the scalar form
+#define GR_VEC_THREADS 512  // of the vector form, at most: a row's loads are then all in flight at once up to 2,048 columns
+#define GR_CHUNKS 4         // four-column groups a thread of the vector form keeps
 
 __device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
 __device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
@@ -98,7 +99,7 @@ __global__ void __launch_bounds__(GR_THREADS) gated_residual_norm_kernel(const G
 }
 
 template <typename TY, typename TA, typename TB, typename TW>
-__global__ void __launch_bounds__(GR_THREADS) gated_residual_norm_vec_kernel(const GatedSum p) {
+__global__ void __launch_bounds__(GR_VEC_THREADS) gated_residual_norm_vec_kernel(const GatedSum p) {
     __shared__ float scratch[32];
     pdl_trigger();
     const int r = blockIdx.x;
@@ -114,7 +115,7 @@ __global__ void __launch_bounds__(GR_THREADS) gated_residual_norm_vec_kernel(con
     float ss = 0.0f;
 #pragma unroll
     for (int c = 0; c < GR_CHUNKS; ++c) {
-        const int i = (c * GR_THREADS + threadIdx.x) * 4;
+        const int i = (c * (int)blockDim.x + threadIdx.x) * 4;
         if (i >= H) break;
         float4 v = load4(xr + i);
         if (values) {
@@ -149,7 +150,7 @@ __global__ void __launch_bounds__(GR_THREADS) gated_residual_norm_vec_kernel(con
     const float inv = w ? rsqrtf(block_sum(ss, scratch) / (float)H + p.eps) : 1.0f;
 #pragma unroll
     for (int c = 0; c < GR_CHUNKS; ++c) {
-        const int i = (c * GR_THREADS + threadIdx.x) * 4;
+        const int i = (c * (int)blockDim.x + threadIdx.x) * 4;
         if (i >= H) break;
         float4 v = kept[c];
         if (w) {
@@ -164,9 +165,11 @@ __global__ void __launch_bounds__(GR_THREADS) gated_residual_norm_vec_kernel(con
 template <typename TY, typename TA>
 static int launch_gated(const GatedSum& p, int R, int bias_bf16, int w_bf16, bool vec, cudaStream_t stream) {
     const size_t smem = vec ? 0 : (size_t)p.H * sizeof(float);
+    const int wanted = (p.H / 4 + 31) / 32 * 32;
+    const int threads = wanted > GR_VEC_THREADS ? GR_VEC_THREADS : wanted;
 #define LAUNCH(TB, TW)                                                                                                          \
     do {                                                                                                                        \
-        if (vec) kb_launch(gated_residual_norm_vec_kernel<TY, TA, TB, TW>, dim3(R), dim3(GR_THREADS), smem, stream, p);           \
+        if (vec) kb_launch(gated_residual_norm_vec_kernel<TY, TA, TB, TW>, dim3(R), dim3(threads), smem, stream, p);              \
         else kb_launch(gated_residual_norm_kernel<TY, TA, TB, TW>, dim3(R), dim3(GR_THREADS), smem, stream, p);                   \
     } while (0)
     if (bias_bf16) {
@@ -188,7 +191,7 @@ KB_EXPORT int kb_gated_residual_norm(float* x, const void* values, int values_bf
     if (out_stride < (origin ? 2 * H : H)) return KB_ERR_BAD_ARG;
     const GatedSum p = {x, values, mix, at, K, extra, gate, gate_stride, bias, mult, w, eps, origin, out, out_stride, rows, H};
     const uintptr_t all = (uintptr_t)x | (uintptr_t)values | (uintptr_t)extra | (uintptr_t)gate | (uintptr_t)bias | (uintptr_t)w | (uintptr_t)origin | (uintptr_t)out;
-    const bool vec = H % 4 == 0 && H <= 4 * GR_CHUNKS * GR_THREADS && gate_stride % 4 == 0 && out_stride % 4 == 0 && all % 16 == 0;
+    const bool vec = H % 4 == 0 && H <= 4 * GR_CHUNKS * GR_VEC_THREADS && gate_stride % 4 == 0 && out_stride % 4 == 0 && all % 16 == 0;
     if (act_bf16) {
         if (values_bf16) return launch_gated<__nv_bfloat16, __nv_bfloat16>(p, R, bias_bf16, w_bf16, vec, stream);
         return launch_gated<float, __nv_bfloat16>(p, R, bias_bf16, w_bf16, vec, stream);

@@ -368,6 +368,8 @@ moe_skinny_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int* __res
     __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(sk_shared);  // [SK_PAIRS][Kp + 32]
     constexpr bool FIRST = FORM != MOE_DOWN;
     constexpr int NB = FORM == MOE_GATED ? 2 : 1;
+    // runs of 32 columns a step: one weight instead of two a lane leaves registers (and needs loads in flight) for twice the run
+    constexpr int RUNS = FORM == MOE_GATED ? 2 : 4, STEP = 32 * RUNS;
     const int ldx = Kp + 32;  // rows fall on alternate halves of a 128-byte line: 16-byte reads of 8 rows do not collide
     pdl_wait();
     const int tile = blockIdx.x;
@@ -407,10 +409,10 @@ moe_skinny_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int* __res
         for (int b = 0; b < NB; ++b)
 #pragma unroll
             for (int c = 0; c < 4; ++c) acc[b][c] = 0.0f;
-        uint4 lo[NB][2], hi[NB][2], nlo[NB][2], nhi[NB][2];
-        auto fetch = [&](int kc, uint4 (&dlo)[NB][2], uint4 (&dhi)[NB][2]) {
+        uint4 lo[NB][RUNS], hi[NB][RUNS], nlo[NB][RUNS], nhi[NB][RUNS];
+        auto fetch = [&](int kc, uint4 (&dlo)[NB][RUNS], uint4 (&dhi)[NB][RUNS]) {
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
+            for (int half = 0; half < RUNS; ++half) {
                 const int col = kc + half * 32 + tg * 8;
 #pragma unroll
                 for (int b = 0; b < NB; ++b) {
@@ -420,10 +422,10 @@ moe_skinny_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int* __res
             }
         };
         fetch(0, lo, hi);
-        for (int kc = 0; kc < Kp; kc += 64) {
-            if (kc + 64 < Kp) fetch(kc + 64, nlo, nhi);
+        for (int kc = 0; kc < Kp; kc += STEP) {
+            if (kc + STEP < Kp) fetch(kc + STEP, nlo, nhi);
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
+            for (int half = 0; half < RUNS; ++half) {
                 const uint4 x = *reinterpret_cast<const uint4*>(xs + (size_t)g * ldx + kc + half * 32 + tg * 8);
                 const uint32_t b0[2] = {x.x, x.y}, b1[2] = {x.z, x.w};
 #pragma unroll
@@ -434,11 +436,11 @@ moe_skinny_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int* __res
                     mma_bf16_16816(acc[b], a1, b1);
                 }
             }
-            if (kc + 64 < Kp) {
+            if (kc + STEP < Kp) {
 #pragma unroll
                 for (int b = 0; b < NB; ++b)
 #pragma unroll
-                    for (int half = 0; half < 2; ++half) {
+                    for (int half = 0; half < RUNS; ++half) {
                         lo[b][half] = nlo[b][half];
                         hi[b][half] = nhi[b][half];
                     }
@@ -680,7 +682,8 @@ KB_EXPORT int kb_moe_skinny(const void* A, int lda, const int* sorted, int top, 
     if (max_tiles == 0) return 0;
     if (!A || !sorted || !W || !tile_expert || !tile_first || !tile_pairs || !num_tiles || !out) return KB_ERR_NULL;
     if (N < 1 || Kd < 8 || top < 1 || Kd % 8 != 0 || lda % 8 != 0 || ((uintptr_t)A % 16) != 0 || ((uintptr_t)W % 16) != 0) return KB_ERR_BAD_ARG;
-    const int Kp = (Kd + 63) / 64 * 64;
+    const int step = form == MOE_GATED ? 64 : 128;  // the kernel's columns a step
+    const int Kp = (Kd + step - 1) / step * step;
     const size_t smem = (size_t)SK_PAIRS * (Kp + 32) * sizeof(__nv_bfloat16);
     if (smem > 200 * 1024) return KB_ERR_UNSUPPORTED_SIZE;
     dim3 grid(max_tiles, (N + SK_FEATURES - 1) / SK_FEATURES);

@@ -7,49 +7,72 @@
 //
 // The H heads are the rows of the products (sixteen a product, as many as a product has anyway), so the wide key row costs no
 // more than G separate heads' keys would, and a request's keys and values are read once for all heads.
-// A block (8 warps) walks a share of one request's keys in tiles of 32 at absolute multiples of 32, first the tiles of the kept
-// first tokens, then the window's, through a ring of cp.async buffers.  Per tile: S, each warp 8 keys and half of the key
-// columns; softmax, a warp a row at a time with a lane a key; P V, each warp its 16-column units of the value row (a unit
-// lies in one key/value head and takes that head's rows of P).  With the keys split over blocks the unnormalised results
-// are combined by a second kernel in split order, so a result depends on the token's position and the number of splits.
+// A block walks a share of one request's keys in tiles of 32 at absolute multiples of 32, first the tiles of the kept first
+// tokens, then the window's.  Four warps copy (cp.async) the tiles' keys and values into a ring of buffers, in the order they are
+// used: K0 K1 V0 K2 V1 ...; eight warps work on them, a turn at a time, in two phases:
+//   products  S of tile n + 1 (warp w: 16 of its keys, a quarter of the key columns, whose part of the queries the warp holds in
+//             registers) and O += P V of tile n (warp w: its 16-column units of the value row; a unit lies in one key/value
+//             head and takes that head's rows of P);
+//   softmax   of tile n + 1, a warp a row, a lane a key: the quarters' scores are added up, the row's maximum moves on, P goes
+//             to shared memory.  A lane keeps its share of the row's sum to itself until the end.
+// With the keys split over blocks the unnormalised results are combined by a second kernel in split order, so a result
+// depends on the token's position and the number of splits.
+// Waits on the ring's barriers are bounded by time: who gives up raises KB_FLAG_TIMEOUT and the block's abort word, later waits end
+// at once, and the block runs to its end over whatever the buffers hold.
 #include "attention_mma.cuh"
 
-#define TD_THREADS 256
-#define TD_WARPS 8
+#define TD_WARPS 8       // that work on the tiles
+#define TD_COPY_WARPS 4  // that fetch them
+#define TD_WORKERS (TD_WARPS * 32)
+#define TD_THREADS ((TD_WARPS + TD_COPY_WARPS) * 32)
+#define TD_MAX_RING 8
+#define TD_IN_FLIGHT 3   // items a copying thread leaves unreported behind the one it has just issued
 #define TD_KEYS 32
 #define TD_P_STRIDE (TD_KEYS + 8)
-#define TD_S_STRIDE (TD_KEYS + 2)
-#define TD_SMEM_LIMIT (220 * 1024)
+#define TD_S_STRIDE (TD_KEYS + 4)
+#define TD_SMEM_LIMIT (226 * 1024)
+
+__device__ __forceinline__ void td_arrive(uint64_t* bar) {
+    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(smem_u32(bar)) : "memory");
+}
+__device__ __forceinline__ bool td_wait(uint64_t* bar, uint32_t parity, volatile int* abort_word) {
+    return !*abort_word && mbar_wait(bar, parity);
+}
 
 struct TdShape {
     int H, G, D, width;  // width = G * D
-    int row_tiles;       // sixteens of query heads
-    int stages;
+    int row_tiles;       // sixteens of query heads: 1 or 2
+    int ring;            // buffers of a tile's keys or values
 };
 
 __host__ __device__ static inline size_t td_smem(const TdShape& s) {
     const size_t stride = s.width + 8, rows = 16 * s.row_tiles;
-    return (rows * stride + (size_t)s.stages * 2 * TD_KEYS * stride + rows * TD_P_STRIDE) * sizeof(__nv_bfloat16)
-           + (2 * rows * TD_S_STRIDE + 3 * rows) * sizeof(float);
+    return ((size_t)s.ring * TD_KEYS * stride + rows * TD_P_STRIDE) * sizeof(__nv_bfloat16) + (4 * rows * TD_S_STRIDE + 3 * rows) * sizeof(float)
+           + 2 * TD_MAX_RING * 8 + 16;
 }
 
-template <int UNITS>  // 16-column units of the value row a warp owns at most
+// MT: sixteens of heads; STEPS: 16-column steps of the key row a warp's quarter has at most (the value row's 16-column units
+// a warp owns are then STEPS / 2 at most)
+template <int MT, int STEPS>
 __global__ void __launch_bounds__(TD_THREADS)
 talking_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfloat16* __restrict__ out, int out_stride,
                       const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ seq_lens,
                       const int* __restrict__ block_table, int max_pages, const int* __restrict__ list_rows,
                       const int* __restrict__ list_tokens, const TdShape shape, int page_size, int page_shift, int num_pages, float scale,
-                      int window, int keep_first, int splits, float* __restrict__ part_o, float* __restrict__ part_ml) {
+                      int window, int keep_first, int splits, float* __restrict__ part_o, float* __restrict__ part_ml, int* flag) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    const int H = shape.H, D = shape.D, width = shape.width, stride = width + 8, rows = 16 * shape.row_tiles, stages = shape.stages;
-    __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem_raw);
-    __nv_bfloat16* sKV = sQ + (size_t)rows * stride;  // per stage: 32 key rows, then 32 value rows
-    const size_t stage_size = (size_t)2 * TD_KEYS * stride;
-    __nv_bfloat16* sP = sKV + stages * stage_size;
-    float* sS = reinterpret_cast<float*>(sP + (size_t)rows * TD_P_STRIDE);  // [column half][row][key]
-    float* sAlpha = sS + 2 * rows * TD_S_STRIDE;
-    float* sM = sAlpha + rows;
-    float* sL = sM + rows;
+    constexpr int UNITS = STEPS / 2, ROWS = 16 * MT, ROW_TURNS = ROWS / TD_WARPS;
+    const int H = shape.H, D = shape.D, width = shape.width, stride = width + 8, ring = shape.ring;
+    const size_t tile_size = (size_t)TD_KEYS * stride;
+    uint64_t* full = reinterpret_cast<uint64_t*>(smem_raw);
+    uint64_t* empty = full + TD_MAX_RING;
+    volatile int* abort_word = reinterpret_cast<volatile int*>(empty + TD_MAX_RING);
+    __nv_bfloat16* sRing = reinterpret_cast<__nv_bfloat16*>(smem_raw + 2 * TD_MAX_RING * 8 + 16);
+    __nv_bfloat16* sP = sRing + ring * tile_size;
+    float* sS = reinterpret_cast<float*>(sP + ROWS * TD_P_STRIDE);  // [column quarter][row][key]
+    float* sAlpha = sS + 4 * ROWS * TD_S_STRIDE;
+    float* sM = sAlpha + ROWS;
+    float* sL = sM + ROWS;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, tq = lane & 3, mm = lane >> 3;
@@ -74,139 +97,244 @@ talking_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bf
         }
         return;
     }
-    const int chunks = width / 8;
-    auto load_tile = [&](int n, int stage) {
-        __nv_bfloat16* tK = sKV + stage * stage_size;
-        __nv_bfloat16* tV = tK + (size_t)TD_KEYS * stride;
-        const int key0 = key_of(n);
-#pragma unroll
-        for (int i = 0; i < TD_KEYS / TD_WARPS; ++i) {
-            const int r = warp + i * TD_WARPS;
-            const int key = key0 + r;
-            bool valid = key <= pos;
-            size_t place = 0;
-            if (valid) {
-                const int page_index = page_shift >= 0 ? key >> page_shift : key / page_size;
-                const int page = page_index < max_pages ? table[page_index] : -1;  // -1: a page the window has given back
-                valid = page >= 0 && page < num_pages;
-                if (valid) place = ((size_t)page * page_size + (key - page_index * page_size)) * width;
-            }
-            for (int c = lane; c < chunks; c += 32) {
-                cp_async16(tK + (size_t)r * stride + c * 8, k_cache + place + (valid ? c * 8 : 0), valid);
-                cp_async16(tV + (size_t)r * stride + c * 8, v_cache + place + (valid ? c * 8 : 0), valid);
-            }
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < ring; ++i) {
+            mbar_init(full + i, TD_COPY_WARPS);
+            mbar_init(empty + i, TD_WARPS);
         }
+        *abort_word = 0;
+        fence_barrier_init();
+    }
+    __syncthreads();
+    auto give_up = [&]() {
+        if (lane == 0 && !*abort_word && flag) atomicOr(flag, KB_FLAG_TIMEOUT);
+        *abort_word = 1;
     };
-    pdl_wait();
-    for (int r = warp; r < rows; r += TD_WARPS)
-        for (int c = lane; c < chunks; c += 32)
-            cp_async16(sQ + (size_t)r * stride + c * 8, q + (size_t)token * q_stride + (r < H ? (size_t)r * width + c * 8 : 0), r < H);
-    // one copy group a tile, also where there is no tile left, so that "all but the last groups" always names the tile at hand
-    for (int ahead = 0; ahead < stages - 1; ++ahead) {
-        if (ahead < num_kt) load_tile(ahead, ahead);
-        cp_async_commit();
-    }
-    for (int r = threadIdx.x; r < rows; r += TD_THREADS) {
-        sM[r] = -INFINITY;
-        sL[r] = 0.0f;
-    }
 
+    if (warp >= TD_WARPS) {
+        // ---------------- copies: a warp takes every fourth row of a tile
+        const int copier = warp - TD_WARPS;
+        constexpr int ROWS_HERE = TD_KEYS / TD_COPY_WARPS;
+        const int chunks = width / 8;
+        int place[ROWS_HERE], place_before[ROWS_HERE];  // where the warp's key rows of a tile lie (in positions of the pool), -1: nowhere
+#pragma unroll
+        for (int i = 0; i < ROWS_HERE; ++i) place[i] = -1;
+        int slot = 0, use = 0, reported = 0, pending = 0;
+        bool ok = true;
+        auto report = [&](int left) {
+            __syncwarp();
+            for (; pending > left; --pending) {
+                if (lane == 0) td_arrive(full + reported);
+                if (++reported == ring) reported = 0;
+            }
+        };
+        auto fetch = [&](const __nv_bfloat16* cache, const int (&at)[ROWS_HERE]) {
+            if (use > 0) {
+                if (!__all_sync(0xffffffffu, mbar_wait(empty + slot, (use - 1) & 1, 1))) {  // report everything issued before waiting: no wait can be circular
+                    cp_async_wait<0>();
+                    report(0);
+                    ok = __all_sync(0xffffffffu, td_wait(empty + slot, (use - 1) & 1, abort_word));
+                    if (!ok) {
+                        give_up();
+                        return;
+                    }
+                }
+            }
+            __nv_bfloat16* tile = sRing + slot * tile_size;
+#pragma unroll
+            for (int i = 0; i < ROWS_HERE; ++i) {
+                const bool valid = at[i] >= 0;
+                const __nv_bfloat16* src = cache + (size_t)(valid ? at[i] : 0) * width;
+                __nv_bfloat16* dst = tile + (size_t)(copier + i * TD_COPY_WARPS) * stride;
+#pragma unroll 2
+                for (int c = lane; c < chunks; c += 32) cp_async16(dst + c * 8, src + c * 8, valid);
+            }
+            cp_async_commit();
+            ++pending;
+            if (++slot == ring) {
+                slot = 0;
+                ++use;
+            }
+            if (pending > TD_IN_FLIGHT) {
+                cp_async_wait<TD_IN_FLIGHT>();
+                report(TD_IN_FLIGHT);
+            }
+        };
+        for (int n = 0; n <= num_kt && ok; ++n) {
+#pragma unroll
+            for (int i = 0; i < ROWS_HERE; ++i) place_before[i] = place[i];
+            if (n < num_kt) {
+                const int key0 = key_of(n);
+#pragma unroll
+                for (int i = 0; i < ROWS_HERE; ++i) {
+                    const int key = key0 + copier + i * TD_COPY_WARPS;
+                    const int page_index = page_shift >= 0 ? key >> page_shift : key / page_size;
+                    const int page = key <= pos && page_index < max_pages ? table[page_index] : -1;  // -1: a page the window has given back
+                    place[i] = page >= 0 && page < num_pages ? page * page_size + (key - page_index * page_size) : -1;
+                }
+                if (n == 0) pdl_wait();  // the pages' numbers do not depend on the kernel before, the newest position's keys do
+                fetch(k_cache, place);
+            }
+            if (n > 0 && ok) fetch(v_cache, place_before);
+        }
+        cp_async_wait<0>();
+        report(0);
+        return;
+    }
+    pdl_wait();
+
+    // ---------------- work
+    auto workers_sync = [&]() { asm volatile("bar.sync 1, %0;\n" ::"n"(TD_WORKERS) : "memory"); };
+    const int steps = width / 16, per_quarter = (steps + 3) / 4;
+    const int key_half = warp & 1, quarter = warp >> 1;
+    const int step0 = quarter * per_quarter, my_steps = max(0, min(per_quarter, steps - step0));
+    // the warp's part of the queries, straight into the products' register layout (rows beyond the heads: zeros)
+    uint32_t qa[MT][STEPS][4];
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int s = 0; s < STEPS; ++s) {
+            const int r0 = mt * 16 + g, col = (step0 + s) * 16 + tq * 2;
+            const __nv_bfloat16* src = q + (size_t)token * q_stride + col;
+            const bool on = s < my_steps;
+            qa[mt][s][0] = on && r0 < H ? *reinterpret_cast<const uint32_t*>(src + (size_t)r0 * width) : 0u;
+            qa[mt][s][1] = on && r0 + 8 < H ? *reinterpret_cast<const uint32_t*>(src + (size_t)(r0 + 8) * width) : 0u;
+            qa[mt][s][2] = on && r0 < H ? *reinterpret_cast<const uint32_t*>(src + (size_t)r0 * width + 8) : 0u;
+            qa[mt][s][3] = on && r0 + 8 < H ? *reinterpret_cast<const uint32_t*>(src + (size_t)(r0 + 8) * width + 8) : 0u;
+        }
     float o[UNITS][2][4];
 #pragma unroll
     for (int u = 0; u < UNITS; ++u)
 #pragma unroll
         for (int t = 0; t < 2; ++t) o[u][t][0] = o[u][t][1] = o[u][t][2] = o[u][t][3] = 0.0f;
-    const int units = width / 16;
-    const int ksteps = width / 16, half_steps = (ksteps + 1) / 2;
-    const int key_group = warp & 3, part = warp >> 2;
-    const int k_begin = part ? half_steps : 0, k_end = part ? ksteps : half_steps;
+    float m_row[ROW_TURNS], l_lane[ROW_TURNS];  // of the rows this warp's softmax takes: warp, warp + 8, ...
+#pragma unroll
+    for (int i = 0; i < ROW_TURNS; ++i) {
+        m_row[i] = -INFINITY;
+        l_lane[i] = 0.0f;
+    }
     const float scale2 = scale * LOG2E;
 
-    int stage = 0;
-    for (int n = 0; n < num_kt; ++n) {
-        if (n + stages - 1 < num_kt) load_tile(n + stages - 1, (stage + stages - 1) % stages);  // the buffer of the tile before
-        cp_async_commit();
-        if (stages == 3) cp_async_wait<2>(); else cp_async_wait<1>();
-        __syncthreads();
-        const __nv_bfloat16* tK = sKV + stage * stage_size;
-        const __nv_bfloat16* tV = tK + (size_t)TD_KEYS * stride;
-        // S: this warp's 8 keys, its half of the key columns, sixteen heads at a time
-        for (int mt = 0; mt < shape.row_tiles; ++mt) {
-            float s[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-            const __nv_bfloat16* q_at = sQ + (size_t)(mt * 16 + (mm & 1) * 8 + (lane & 7)) * stride + (mm >> 1) * 8;
-            const __nv_bfloat16* k_at = tK + (size_t)(key_group * 8 + (lane & 7)) * stride + mm * 8;
-#pragma unroll 4
-            for (int ks = k_begin; ks < k_end; ks += 2) {
-                uint32_t a[4], b[4];
-                ldmatrix_x4(b, k_at + ks * 16);  // the keys' columns of two steps
-                ldmatrix_x4(a, q_at + ks * 16);
-                mma_16816(s, a, b[0], b[1]);
-                if (ks + 1 < k_end) {
-                    ldmatrix_x4(a, q_at + ks * 16 + 16);
-                    mma_16816(s, a, b[2], b[3]);
+    int head_of_unit[UNITS];  // the first query head of the unit's key/value head
+#pragma unroll
+    for (int u = 0; u < UNITS; ++u) head_of_unit[u] = ((warp + u * TD_WARPS) * 16 / D) * group;
+
+    int slot = 0, use = 0;  // of the next item
+    auto item_ready = [&]() {
+        if (!td_wait(full + slot, use & 1, abort_word)) give_up();
+        __syncwarp();
+        return sRing + slot * tile_size;
+    };
+    auto item_done = [&]() {
+        __syncwarp();
+        if (lane == 0) td_arrive(empty + slot);
+        if (++slot == ring) {
+            slot = 0;
+            ++use;
+        }
+    };
+    for (int t = 0; t <= num_kt; ++t) {
+        if (t < num_kt) {
+            const __nv_bfloat16* k_at = item_ready() + (size_t)(key_half * 16 + (mm >> 1) * 8 + (lane & 7)) * stride + (size_t)step0 * 16 + (mm & 1) * 8;
+            float s[MT][2][4];
+#pragma unroll
+            for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+                for (int x = 0; x < 2; ++x) s[mt][x][0] = s[mt][x][1] = s[mt][x][2] = s[mt][x][3] = 0.0f;
+#pragma unroll
+            for (int ks = 0; ks < STEPS; ++ks) {
+                if (ks >= my_steps) break;
+                uint32_t b[4];
+                ldmatrix_x4(b, k_at + ks * 16);
+#pragma unroll
+                for (int mt = 0; mt < MT; ++mt) {
+                    mma_16816(s[mt][0], qa[mt][ks], b[0], b[1]);
+                    mma_16816(s[mt][1], qa[mt][ks], b[2], b[3]);
                 }
             }
-            float* dst = sS + ((size_t)part * rows + mt * 16 + g) * TD_S_STRIDE + key_group * 8 + tq * 2;
-            *reinterpret_cast<float2*>(dst) = make_float2(s[0], s[1]);
-            *reinterpret_cast<float2*>(dst + 8 * TD_S_STRIDE) = make_float2(s[2], s[3]);
+#pragma unroll
+            for (int mt = 0; mt < MT; ++mt) {
+                float* dst = sS + (size_t)(quarter * ROWS + mt * 16 + g) * TD_S_STRIDE + key_half * 16 + tq * 2;
+#pragma unroll
+                for (int x = 0; x < 2; ++x) {
+                    *reinterpret_cast<float2*>(dst + x * 8) = make_float2(s[mt][x][0], s[mt][x][1]);
+                    *reinterpret_cast<float2*>(dst + 8 * TD_S_STRIDE + x * 8) = make_float2(s[mt][x][2], s[mt][x][3]);
+                }
+            }
+            item_done();
         }
-        __syncthreads();
-        // softmax: a warp a row, a lane a key
-        {
-            const int key = key_of(n) + lane;
+        if (t > 0) {
+            const __nv_bfloat16* tV = item_ready();
+#pragma unroll
+            for (int u = 0; u < UNITS; ++u) {
+                const int unit = warp + u * TD_WARPS;
+                if (unit >= steps) break;
+                const int head0 = head_of_unit[u];
+                const float alpha0 = sAlpha[min(head0 + g, H - 1)], alpha1 = sAlpha[min(head0 + g + 8, H - 1)];
+#pragma unroll
+                for (int x = 0; x < 2; ++x) {
+                    o[u][x][0] *= alpha0;
+                    o[u][x][1] *= alpha0;
+                    o[u][x][2] *= alpha1;
+                    o[u][x][3] *= alpha1;
+                }
+                // rows beyond the group hold other heads' weights: their results are dropped
+                const __nv_bfloat16* p_at = sP + (size_t)min(head0 + (mm & 1) * 8 + (lane & 7), H - 1) * TD_P_STRIDE + (mm >> 1) * 8;
+#pragma unroll
+                for (int kk = 0; kk < TD_KEYS / 16; ++kk) {
+                    uint32_t a[4], b[4];
+                    ldmatrix_x4(a, p_at + kk * 16);
+                    ldmatrix_x4_trans(b, tV + (size_t)(kk * 16 + (mm & 1) * 8 + (lane & 7)) * stride + unit * 16 + (mm >> 1) * 8);
+                    mma_16816(o[u][0], a, b[0], b[1]);
+                    mma_16816(o[u][1], a, b[2], b[3]);
+                }
+            }
+            item_done();
+        }
+        workers_sync();
+        if (t < num_kt) {
+            const int key = key_of(t) + lane;
             const bool seen = key <= pos && (key >= key_lo || key < keep_first);
-            for (int r = warp; r < H; r += TD_WARPS) {
-                const float raw = (sS[(size_t)r * TD_S_STRIDE + lane] + sS[((size_t)rows + r) * TD_S_STRIDE + lane]) * scale2;
-                const float value = seen ? raw : -INFINITY;
-                const float before = sM[r];
-                const float top = fmaxf(before, warp_max(value));
-                const float base = top == -INFINITY ? 0.0f : top;
-                const float p = exp2f(value - base);
-                const float alpha = exp2f(before - base);
-                const float sum = warp_sum(p);
-                sP[(size_t)r * TD_P_STRIDE + lane] = __float2bfloat16_rn(p);
-                __syncwarp();
-                if (lane == 0) {
-                    sM[r] = top;
-                    sL[r] = sL[r] * alpha + sum;
-                    sAlpha[r] = alpha;
-                }
+            float value[ROW_TURNS], top[ROW_TURNS];
+#pragma unroll
+            for (int i = 0; i < ROW_TURNS; ++i) {
+                const float* src = sS + (size_t)(warp + i * TD_WARPS) * TD_S_STRIDE + lane;
+                const float raw = (src[0] + src[ROWS * TD_S_STRIDE]) + (src[2 * ROWS * TD_S_STRIDE] + src[3 * ROWS * TD_S_STRIDE]);
+                value[i] = seen ? raw * scale2 : -INFINITY;
+                top[i] = value[i];
+            }
+#pragma unroll
+            for (int offset = 16; offset > 0; offset >>= 1)
+#pragma unroll
+                for (int i = 0; i < ROW_TURNS; ++i) top[i] = fmaxf(top[i], __shfl_xor_sync(0xffffffffu, top[i], offset));
+#pragma unroll
+            for (int i = 0; i < ROW_TURNS; ++i) {
+                const int r = warp + i * TD_WARPS;
+                const float m_new = fmaxf(m_row[i], top[i]);
+                const float base = m_new == -INFINITY ? 0.0f : m_new;
+                const float p = exp2f(value[i] - base);
+                const float alpha = exp2f(m_row[i] - base);
+                l_lane[i] = l_lane[i] * alpha + p;
+                m_row[i] = m_new;
+                sP[r * TD_P_STRIDE + lane] = __float2bfloat16_rn(p);
+                if (lane == 0) sAlpha[r] = alpha;
             }
         }
-        __syncthreads();
-        // O: this warp's units of the value row
-#pragma unroll
-        for (int u = 0; u < UNITS; ++u) {
-            const int unit = warp + u * TD_WARPS;
-            if (unit >= units) break;
-            const int head0 = (unit * 16 / D) * group;  // the first query head of the unit's key/value head
-            const float alpha0 = sAlpha[min(head0 + g, H - 1)], alpha1 = sAlpha[min(head0 + g + 8, H - 1)];
-#pragma unroll
-            for (int t = 0; t < 2; ++t) {
-                o[u][t][0] *= alpha0;
-                o[u][t][1] *= alpha0;
-                o[u][t][2] *= alpha1;
-                o[u][t][3] *= alpha1;
-            }
-            // rows beyond the group hold other heads' weights: their results are dropped
-            const __nv_bfloat16* p_at = sP + (size_t)min(head0 + (mm & 1) * 8 + (lane & 7), H - 1) * TD_P_STRIDE + (mm >> 1) * 8;
-#pragma unroll
-            for (int kk = 0; kk < TD_KEYS / 16; ++kk) {
-                uint32_t a[4], b[4];
-                ldmatrix_x4(a, p_at + kk * 16);
-                ldmatrix_x4_trans(b, tV + (size_t)(kk * 16 + (mm & 1) * 8 + (lane & 7)) * stride + unit * 16 + (mm >> 1) * 8);
-                mma_16816(o[u][0], a, b[0], b[1]);
-                mma_16816(o[u][1], a, b[2], b[3]);
-            }
-        }
-        __syncthreads();  // the buffer is refilled by the next turn's request
-        stage = (stage + 1) % stages;
+        workers_sync();
     }
-    cp_async_wait<0>();
+#pragma unroll
+    for (int i = 0; i < ROW_TURNS; ++i) {
+        const float sum = warp_sum(l_lane[i]);
+        if (lane == 0) {
+            sM[warp + i * TD_WARPS] = m_row[i];
+            sL[warp + i * TD_WARPS] = sum;
+        }
+    }
+    workers_sync();
 #pragma unroll
     for (int u = 0; u < UNITS; ++u) {
         const int unit = warp + u * TD_WARPS;
-        if (unit >= units) break;
+        if (unit >= steps) break;
         const int c = unit * 16 / D, col = unit * 16 - c * D + tq * 2;
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
@@ -216,18 +344,18 @@ talking_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bf
             if (splits > 1) {
                 float* dst = part_o + (((size_t)split * gridDim.y + index) * H + h) * D + col;
 #pragma unroll
-                for (int t = 0; t < 2; ++t) *reinterpret_cast<float2*>(dst + t * 8) = make_float2(o[u][t][half * 2], o[u][t][half * 2 + 1]);
+                for (int x = 0; x < 2; ++x) *reinterpret_cast<float2*>(dst + x * 8) = make_float2(o[u][x][half * 2], o[u][x][half * 2 + 1]);
             } else {
                 const float inv = sL[h] > 0.0f ? 1.0f / sL[h] : 0.0f;
                 __nv_bfloat16* dst = out + (size_t)token * out_stride + (size_t)h * D + col;
 #pragma unroll
-                for (int t = 0; t < 2; ++t)
-                    *reinterpret_cast<__nv_bfloat162*>(dst + t * 8) = __floats2bfloat162_rn(o[u][t][half * 2] * inv, o[u][t][half * 2 + 1] * inv);
+                for (int x = 0; x < 2; ++x)
+                    *reinterpret_cast<__nv_bfloat162*>(dst + x * 8) = __floats2bfloat162_rn(o[u][x][half * 2] * inv, o[u][x][half * 2 + 1] * inv);
             }
         }
     }
     if (splits > 1)
-        for (int h = threadIdx.x; h < H; h += TD_THREADS) {
+        for (int h = threadIdx.x; h < H; h += TD_WORKERS) {
             float* ml = part_ml + (((size_t)split * gridDim.y + index) * H + h) * 2;
             ml[0] = sM[h];
             ml[1] = sL[h];
@@ -260,10 +388,9 @@ talking_decode_merge_kernel(const float* __restrict__ part_o, const float* __res
 }
 
 static bool td_shape(int H, int G, int D, TdShape* shape) {
-    if (G < 1 || H < 1 || H % G != 0 || H / G > 16 || H > 64 || D < 16 || D % 16 != 0 || G * D > 16 * TD_WARPS * 8) return false;
-    TdShape s = {H, G, D, G * D, (H + 15) / 16, 3};
-    if (td_smem(s) > TD_SMEM_LIMIT) s.stages = 2;
-    if (td_smem(s) > TD_SMEM_LIMIT) return false;
+    if (G < 1 || H < 1 || H % G != 0 || H / G > 16 || H > 32 || D < 16 || D % 16 != 0 || G * D > 512) return false;
+    TdShape s = {H, G, D, G * D, (H + 15) / 16, TD_MAX_RING};
+    while (td_smem(s) > TD_SMEM_LIMIT) --s.ring;  // six at the widest row
     *shape = s;
     return true;
 }
@@ -284,45 +411,57 @@ KB_EXPORT int kb_talking_decode_splits(int count, int keys, int H, int G, int D)
     }
     if (count < 1 || !td_shape(H, G, D, &shape)) return 1;
     const int resident = (int)((227 * 1024) / (td_smem(shape) + 1024));
-    const int places = sms * (resident < 1 ? 1 : resident > 4 ? 4 : resident);
+    const int places = sms * (resident < 1 ? 1 : resident > 2 ? 2 : resident);
     const int tiles = (keys + TD_KEYS - 1) / TD_KEYS;
     int splits = places / count;
     if (splits > tiles / 2) splits = tiles / 2;
     return splits < 1 ? 1 : splits > 64 ? 64 : splits;
 }
 
+template <int MT, int STEPS>
+static void launch_decode(size_t smem, cudaStream_t stream, const void* q, int q_stride, void* out, int out_stride, const void* k_cache,
+                          const void* v_cache, const int* seq_lens, const int* block_table, int max_pages, const int* list_rows,
+                          const int* list_tokens, const TdShape& shape, int count, int page_size, int shift, int num_pages, float scale,
+                          int window, int keep_first, int splits, float* part_o, float* part_ml, int* flag) {
+    static bool configured = false;
+    if (!configured) {
+        cudaFuncSetAttribute(talking_decode_kernel<MT, STEPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, TD_SMEM_LIMIT);
+        configured = true;
+    }
+    kb_launch(talking_decode_kernel<MT, STEPS>, dim3(splits, count), dim3(TD_THREADS), smem, stream, (const __nv_bfloat16*)q, q_stride,
+              (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, seq_lens, block_table, max_pages,
+              list_rows, list_tokens, shape, page_size, shift, num_pages, scale, window, keep_first, splits, part_o, part_ml, flag);
+}
+
 KB_EXPORT int kb_talking_decode(const void* q, int q_stride, void* out, int out_stride, const void* k_cache, const void* v_cache,
                                 const int* seq_lens, const int* block_table, int max_pages, const int* list_rows, const int* list_tokens,
                                 int count, int H, int G, int D, int page_size, int num_pages, float scale, int window, int keep_first,
-                                int splits, float* part_o, float* part_ml, cudaStream_t stream) {
+                                int splits, float* part_o, float* part_ml, int* flag, cudaStream_t stream) {
     if (count == 0) return 0;
     if (!q || !out || !k_cache || !v_cache || !seq_lens || !block_table || !list_rows || !list_tokens || (splits > 1 && (!part_o || !part_ml))) return KB_ERR_NULL;
     TdShape shape;
     if (!td_shape(H, G, D, &shape)) return KB_ERR_UNSUPPORTED_SIZE;
     if (count > 65535 || splits < 1 || page_size < 1 || keep_first < 0 || q_stride % 8 || out_stride % 2
         || (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache) % 16) || ((uintptr_t)out % 4)) return KB_ERR_BAD_ARG;
+    if ((long long)num_pages * page_size > 0x7fffffffLL) return KB_ERR_UNSUPPORTED_SIZE;
     const size_t smem = td_smem(shape);
     int shift = -1;
     if ((page_size & (page_size - 1)) == 0) {
         shift = 0;
         while ((1 << shift) < page_size) ++shift;
     }
-#define LAUNCH(U)                                                                                                                             \
-    do {                                                                                                                                      \
-        static bool configured = false;                                                                                                       \
-        if (!configured) {                                                                                                                    \
-            cudaFuncSetAttribute(talking_decode_kernel<U>, cudaFuncAttributeMaxDynamicSharedMemorySize, TD_SMEM_LIMIT);                         \
-            configured = true;                                                                                                                \
-        }                                                                                                                                     \
-        kb_launch(talking_decode_kernel<U>, dim3(splits, count), dim3(TD_THREADS), smem, stream, (const __nv_bfloat16*)q, q_stride,            \
-                  (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, seq_lens, block_table,         \
-                  max_pages, list_rows, list_tokens, shape, page_size, shift, num_pages, scale, window, keep_first, splits,       \
-                  part_o, part_ml);                                                                                                           \
-    } while (0)
-    const int per_warp = (shape.width / 16 + TD_WARPS - 1) / TD_WARPS;
-    if (per_warp <= 2) LAUNCH(2);
-    else if (per_warp <= 4) LAUNCH(4);
-    else LAUNCH(8);
+#define LAUNCH(MT, STEPS)                                                                                                                  \
+    launch_decode<MT, STEPS>(smem, stream, q, q_stride, out, out_stride, k_cache, v_cache, seq_lens, block_table, max_pages, list_rows,      \
+                             list_tokens, shape, count, page_size, shift, num_pages, scale, window, keep_first, splits, part_o, part_ml, flag)
+    if (shape.row_tiles == 1) {
+        if (shape.width <= 128) LAUNCH(1, 2);
+        else if (shape.width <= 256) LAUNCH(1, 4);
+        else LAUNCH(1, 8);
+    } else {
+        if (shape.width <= 128) LAUNCH(2, 2);
+        else if (shape.width <= 256) LAUNCH(2, 4);
+        else LAUNCH(2, 8);
+    }
 #undef LAUNCH
     if (splits > 1)
         kb_launch(talking_decode_merge_kernel, dim3(count, H), dim3(128), 0, stream, (const float*)part_o, (const float*)part_ml, (__nv_bfloat16*)out,

@@ -9,36 +9,39 @@
 //
 // A block takes 128 / (H / G) queries of one key/value head: row r of its tile is query r / (H / G), head r % (H / G) of that
 // key/value head's query heads, so the 128 rows of every product share one pass over keys and values.  Keys go in tiles of
-// 128 at absolute multiples of 128: first the tiles of the kept first tokens, then those of the window.  Roles (256 threads; eight warps, so
-// that a thread may hold its 128 scores in registers):
-//   warps 0-3  softmax: thread r owns row r; reads its row of S from tensor memory, writes P as bf16 pairs over it, rescales O
-//              in tensor memory only when the row maximum has grown by more than 2^8 since the reference it scales by;
-//   warps 4-5  producer: cp.async of the queries (once), of the keys, one 64-column band of a tile at a time through a ring of
-//              buffers, and of the values (one buffer), each 16-byte group put where the 128-byte swizzle of the tensor cores'
-//              operand wants it.  (A TMA copy brings a page's run of rows of one band: with pages of 16 positions and wide
-//              keys that is 8 copies for every 256 cycles of products, more than an SM can issue; a thread's cp.async takes
-//              any page size, and pads columns up to 64 and rows beyond the last key with zeros.)
-//   warp 6     one thread issues tcgen05.mma: S (128 x 128, two buffers) band by band, O += P V.  Q K^T runs two tiles
-//              ahead of P V.
-// The items (bands of keys, tiles of values) are produced in the order the products consume them, K0 K1 V0 K2 V1 ..., and a
-// producer thread that has to wait for a free buffer first reports everything it has issued, so no wait can be circular.
+// 64 at absolute multiples of 64: first the tiles of the kept first tokens, then those of the window.  The queries live in
+// tensor memory (two bf16 columns a 32-bit one: 256 of its 512 columns for key rows of 512), which leaves the whole shared
+// memory to the keys and values on their way.  Roles (288 threads):
+//   warps 0-3  softmax: thread r owns row r; moves its queries from shared memory (where they lie in the keys' buffers before
+//              the first keys do) into tensor memory, then reads its row of S from there, writes P as bf16 pairs over it, and
+//              rescales O in tensor memory only when the row maximum has grown by more than 2^8 since the reference it scales by;
+//   warps 4-7  producer: cp.async of a tile's keys or values into its buffer, each 16-byte group put where the 128-byte swizzle
+//              of the tensor cores' operand wants it.  (A TMA copy brings a page's run of rows of one 64-column band: with pages
+//              of 16 positions and wide keys that is 32 copies a tile beside those of the values, more than an SM can issue
+//              beside the products; a thread's cp.async takes any page size, and pads columns up to 64 and rows beyond the
+//              last key with zeros.)
+//   warp 8     one thread issues tcgen05.mma: S (128 x 64, two buffers), O += P V.  Q K^T runs two tiles ahead of P V.
+// A buffer holds a whole tile: with a barrier for every band of a tile the issuing thread spent 540 cycles a band of four
+// products on waiting and committing, three times what the products take.
+// The items are produced in the order the products consume them, K0 K1 V0 K2 V1 ..., and a producer warp that has to wait
+// for a free buffer first reports everything it has issued, so no wait can be circular.
 //
 // Every wait on an mbarrier is bounded: a role that gives up raises KB_FLAG_TIMEOUT, the other roles leave through a shared
 // abort word, and the block frees its tensor memory and returns.
-// Sizes: D a multiple of 8 up to 128, G * D up to 640, H / G up to 128, any page size.
+// Sizes: D a multiple of 8 up to 128, G * D up to 512, H / G up to 128, any page size.
 #include "umma.cuh"
 
-#define TA_THREADS 256
-#define TA_PRODUCERS 64
-#define TA_PASSES (TA_BN * 8 / TA_PRODUCERS)  // rows of a band a producer thread copies 16 bytes of
+#define TA_THREADS 288
+#define TA_PRODUCERS 128
 #define TA_BM 128
-#define TA_BN 128
-#define TA_BAND (TA_BN * 128)  // bytes of one 64-column band of 128 rows
-#define TA_MAX_STAGES 8
+#define TA_BN 64
+#define TA_BAND (TA_BN * 128)  // bytes of one 64-column band of 64 rows
+#define TA_PASSES (TA_BN * 8 / TA_PRODUCERS)  // rows of a band a producer thread copies 16 bytes of
+#define TA_MAX_BANDS 8
+#define TA_K_STAGES 3          // the queries lie in the last two of them before the second tile's keys do
+#define TA_V_STAGES 2
 #define TA_LOG2E 1.4426950408889634f
 #define TA_RESCALE_STEP 8.0f
-#define TA_S_COL 0      // two S buffers of 128 columns; P (bf16 pairs) overwrites the first half of its S
-#define TA_O_COL 256
 #define TA_TMEM_COLUMNS 512
 #define KB_FLAG_MISALIGNED 32
 
@@ -49,7 +52,7 @@ __device__ __forceinline__ float ta_ex2(float x) {
 }
 __device__ __forceinline__ bool ta_ready(uint64_t* bar, uint32_t parity) {
     uint32_t done;
-    asm volatile("{\n .reg .pred p;\n mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n selp.u32 %0, 1, 0, p;\n}\n"
+    asm volatile("{\n .reg .pred p;\n mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n selp.u32 %0, 1, 0, p;\n}\n"
                  : "=r"(done)
                  : "r"(smem_addr(bar)), "r"(parity)
                  : "memory");
@@ -63,65 +66,46 @@ __device__ __forceinline__ void ta_commit() { asm volatile("cp.async.commit_grou
 template <int N>
 __device__ __forceinline__ void ta_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
 
-// A producer thread's items in flight: reported (fence, then one arrival) in the order they were issued.
-struct TaInFlight {
-    uint64_t* older = nullptr;
-    uint64_t* newer = nullptr;
-    __device__ __forceinline__ void flush() {
-        if (!newer) return;
-        ta_wait<0>();
-        fence_proxy_async_smem();
-        if (older) mbar_arrive(older);
-        mbar_arrive(newer);
-        older = newer = nullptr;
-    }
-    __device__ __forceinline__ void push(uint64_t* bar) {  // the copies issued since the last push belong to `bar`
-        ta_commit();
-        if (older) {  // two items stay in flight behind this one
-            ta_wait<2>();
-            fence_proxy_async_smem();
-            mbar_arrive(older);
-        }
-        older = newer;
-        newer = bar;
-    }
-};
-
 template <int VB>  // 64-column bands of a value row
 __global__ void __launch_bounds__(TA_THREADS, 1)
 talking_attention_tc5_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfloat16* __restrict__ out, int out_stride,
                              const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
                              const int* __restrict__ qo_indptr, const int* __restrict__ seq_lens, const int* __restrict__ block_table,
                              int max_pages, const int* __restrict__ tile_rows, const int* __restrict__ tile_starts, int H, int G, int D,
-                             int key_bands, int stages, int page_size, int page_shift, int num_pages, float scale, int window,
+                             int key_bands, int page_size, int page_shift, int num_pages, float scale, int window,
                              int keep_first, int* flag) {
     extern __shared__ __align__(1024) unsigned char smem[];
-    unsigned char* sQ = smem;
-    unsigned char* sK = sQ + (size_t)key_bands * TA_BAND;
-    unsigned char* sV = sK + (size_t)stages * TA_BAND;
-    uint64_t* bars = reinterpret_cast<uint64_t*>(sV + VB * TA_BAND);
-    uint64_t* q_full = bars;
-    uint64_t* k_full = bars + 1;
-    uint64_t* k_empty = k_full + TA_MAX_STAGES;
-    uint64_t* v_full = k_empty + TA_MAX_STAGES;
-    uint64_t* v_empty = v_full + 1;
-    uint64_t* s_full = v_empty + 1;   // one per S buffer
+    const uint32_t k_bytes = key_bands * TA_BAND, v_bytes = VB * TA_BAND;
+    unsigned char* sV = smem + TA_K_STAGES * k_bytes;
+    uint64_t* bars = reinterpret_cast<uint64_t*>(sV + TA_V_STAGES * v_bytes);
+    uint64_t* k_full = bars;
+    uint64_t* k_empty = k_full + TA_K_STAGES;
+    uint64_t* v_full = k_empty + TA_K_STAGES;
+    uint64_t* v_empty = v_full + TA_V_STAGES;
+    uint64_t* q_loaded = v_empty + TA_V_STAGES;  // the queries lie in shared memory
+    uint64_t* q_stored = q_loaded + 1;           // ... and in tensor memory
+    uint64_t* s_full = q_stored + 1;             // one per S buffer
     // two each, used in turn: the softmax may be a tile ahead of the products, and a barrier whose phase is told by its
     // parity cannot be two phases ahead of who waits on it
     uint64_t* p_full = s_full + 2;
     uint64_t* pv_done = p_full + 2;
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 2);
     volatile int* abort_word = reinterpret_cast<volatile int*>(tmem_slot + 1);
+    // tensor memory: two S buffers of 64 columns (P, bf16 pairs, overwrites the first half of its S), O, the queries
+    constexpr int S_COL = 0, O_COL = 2 * TA_BN, Q_COL = O_COL + VB * 64;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
-        mbar_init(q_full, TA_PRODUCERS);
-        for (int s = 0; s < stages; ++s) {
-            mbar_init(k_full + s, TA_PRODUCERS);
+        for (int s = 0; s < TA_K_STAGES; ++s) {
+            mbar_init(k_full + s, TA_PRODUCERS / 32);
             mbar_init(k_empty + s, 1);
         }
-        mbar_init(v_full, TA_PRODUCERS);
-        mbar_init(v_empty, 1);
+        for (int s = 0; s < TA_V_STAGES; ++s) {
+            mbar_init(v_full + s, TA_PRODUCERS / 32);
+            mbar_init(v_empty + s, 1);
+        }
+        mbar_init(q_loaded, TA_PRODUCERS / 32);
+        mbar_init(q_stored, 4);
         for (int i = 0; i < 2; ++i) {
             mbar_init(s_full + i, 1);
             mbar_init(p_full + i, 4);
@@ -135,7 +119,7 @@ talking_attention_tc5_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, 
         asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
         fence_proxy_async_smem();
     }
-    if (warp == 6) tmem_alloc(tmem_slot, TA_TMEM_COLUMNS);
+    if (warp == 8) tmem_alloc(tmem_slot, TA_TMEM_COLUMNS);
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
@@ -162,43 +146,73 @@ talking_attention_tc5_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, 
 
     if (*abort_word || num_kt == 0) {
         // fall through to the common exit
-    } else if (warp == 4 || warp == 5) {
-        // ---------------- producer: 8 lanes a row, 8 rows a pass
+    } else if (warp >= 4 && warp < 8) {
+        // ---------------- producer: 8 lanes a row, 16 rows a pass
         const int tid = threadIdx.x - 128;
         const int chunk = tid & 7, row0 = tid >> 3;
         const int key_width = G * D;
-        const uint32_t swizzled = (uint32_t)((chunk ^ (row0 & 7)) * 16);  // rows of a thread differ by 8: one swizzle for all
+        const uint32_t row_at = smem_addr(smem) + row0 * 128 + (uint32_t)((chunk ^ (row0 & 7)) * 16);  // a thread's rows are 16 apart: one swizzle
+        const uint32_t v_at = row_at + TA_K_STAGES * k_bytes;
         const int* table = block_table + (size_t)row * max_pages;
-        TaInFlight flight;
         bool ok = true;
-        auto wait_free = [&](uint64_t* bar, uint32_t parity) {
-            if (ta_ready(bar, parity)) return true;
-            flight.flush();
-            if (mbar_wait(bar, parity, abort_word)) return true;
-            if (!*abort_word && flag) atomicOr(flag, KB_FLAG_TIMEOUT);
-            *abort_word = 1;
-            return false;
+        uint64_t* older = nullptr;  // the barriers of the last two items issued, not reported yet
+        uint64_t* newer = nullptr;
+        auto report = [&](uint64_t* bar) {  // one arrival a warp
+            __syncwarp();
+            if (lane == 0 && bar) mbar_arrive(bar);
         };
-        for (int b = 0; b < key_bands; ++b) {
-            const int col = b * 64 + chunk * 8;
-#pragma unroll
-            for (int i = 0; i < TA_PASSES; ++i) {
-                const int r = row0 + i * 8;
-                const int qi = r / group;
-                const bool valid = qi < queries && col < key_width;
-                const __nv_bfloat16* src = q + (size_t)(tok0 + q0 + (valid ? qi : 0)) * q_stride + (size_t)(kvh * group + (valid ? r - qi * group : 0)) * key_width + (valid ? col : 0);
-                ta_copy16(smem_addr(sQ) + b * TA_BAND + r * 128 + swizzled, src, valid);
+        auto flush = [&]() {
+            ta_wait<0>();
+            fence_proxy_async_smem();
+            report(older);
+            report(newer);
+            older = newer = nullptr;
+        };
+        auto wait_free = [&](uint64_t* bar, uint32_t parity) {
+            if (__all_sync(0xffffffffu, ta_ready(bar, parity))) return true;
+            flush();
+            ok = __all_sync(0xffffffffu, mbar_wait(bar, parity, abort_word));
+            if (!ok) {
+                if (lane == 0 && !*abort_word && flag) atomicOr(flag, KB_FLAG_TIMEOUT);
+                *abort_word = 1;
+            }
+            return ok;
+        };
+        auto end_item = [&](uint64_t* bar) {  // the copies issued since the last call belong to `bar`
+            ta_commit();
+            if (older) {
+                ta_wait<2>();
+                fence_proxy_async_smem();
+                report(older);
+            }
+            older = newer;
+            newer = bar;
+        };
+        // the queries: row r at r * bands * 128 bytes behind the first keys' buffer, a band's 16-byte groups turned by the row
+        for (int r = row0; r < TA_BM; r += 16) {
+            const int qi = r / group;
+            const bool in_tile = qi < queries && r < per_tile * group;
+            const __nv_bfloat16* src = q + (size_t)(tok0 + q0 + (in_tile ? qi : 0)) * q_stride + (size_t)(kvh * group + (in_tile ? r - qi * group : 0)) * key_width;
+            const uint32_t dst = smem_addr(smem) + k_bytes + r * key_bands * 128 + (uint32_t)((chunk ^ (r & 7)) * 16);
+            for (int b = 0; b < key_bands; ++b) {
+                const int col = b * 64 + chunk * 8;
+                const bool valid = in_tile && col < key_width;
+                ta_copy16(dst + b * 128, src + (valid ? col : 0), valid);
             }
         }
-        flight.push(q_full);
+        end_item(q_loaded);
         int place[TA_PASSES], place_before[TA_PASSES];
-        uint32_t slot = 0, use = 0;  // of the key ring
+#pragma unroll
+        for (int i = 0; i < TA_PASSES; ++i) place[i] = -1;
+        int k_slot = 0, k_use = 0;
         for (int n = 0; n <= num_kt && ok; ++n) {
+#pragma unroll
+            for (int i = 0; i < TA_PASSES; ++i) place_before[i] = place[i];
             if (n < num_kt) {
                 const int key0 = key_of(n);
 #pragma unroll
                 for (int i = 0; i < TA_PASSES; ++i) {
-                    const int key = key0 + row0 + i * 8;
+                    const int key = key0 + row0 + i * 16;
                     int at = -1;
                     if (key < key_end) {
                         const int page_index = page_shift >= 0 ? key >> page_shift : key / page_size;
@@ -207,96 +221,91 @@ talking_attention_tc5_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, 
                     }
                     place[i] = at;
                 }
+                if (n == 1 && !wait_free(q_stored, 0)) break;  // the queries have left the buffers of the tiles after the first
+                if (k_use > 0 && !wait_free(k_empty + k_slot, (k_use - 1) & 1)) break;
                 for (int b = 0; b < key_bands; ++b) {
-                    if (use > 0 && !wait_free(k_empty + slot, (use - 1) & 1)) {
-                        ok = false;
-                        break;
-                    }
                     const int col = b * 64 + chunk * 8;
-                    const uint32_t dst = smem_addr(sK) + slot * TA_BAND + row0 * 128 + swizzled;
 #pragma unroll
                     for (int i = 0; i < TA_PASSES; ++i) {
                         const bool valid = place[i] >= 0 && col < key_width;
-                        ta_copy16(dst + i * 1024, k_cache + (valid ? (size_t)place[i] * key_width + col : 0), valid);
+                        ta_copy16(row_at + k_slot * k_bytes + b * TA_BAND + i * 2048, k_cache + (valid ? (size_t)place[i] * key_width + col : 0), valid);
                     }
-                    flight.push(k_full + slot);
-                    if (++slot == (uint32_t)stages) {
-                        slot = 0;
-                        ++use;
-                    }
+                }
+                end_item(k_full + k_slot);
+                if (++k_slot == TA_K_STAGES) {
+                    k_slot = 0;
+                    ++k_use;
                 }
             }
-            if (n > 0 && ok) {  // the values of the tile before
-                if (n > 1 && !wait_free(v_empty, (n - 2) & 1)) {
-                    ok = false;
-                    break;
-                }
+            if (n > 0) {  // the values of the tile before
+                const int m = n - 1, v_slot = m % TA_V_STAGES;
+                if (m >= TA_V_STAGES && !wait_free(v_empty + v_slot, (m / TA_V_STAGES - 1) & 1)) break;
 #pragma unroll
                 for (int b = 0; b < VB; ++b) {
                     const int col = b * 64 + chunk * 8;
-                    const uint32_t dst = smem_addr(sV) + b * TA_BAND + row0 * 128 + swizzled;
 #pragma unroll
                     for (int i = 0; i < TA_PASSES; ++i) {
                         const bool valid = place_before[i] >= 0 && col < D;
-                        ta_copy16(dst + i * 1024, v_cache + (valid ? (size_t)place_before[i] * key_width + kvh * D + col : 0), valid);
+                        ta_copy16(v_at + v_slot * v_bytes + b * TA_BAND + i * 2048, v_cache + (valid ? (size_t)place_before[i] * key_width + kvh * D + col : 0), valid);
                     }
                 }
-                flight.push(v_full);
+                end_item(v_full + v_slot);
             }
-#pragma unroll
-            for (int i = 0; i < TA_PASSES; ++i) place_before[i] = place[i];
         }
-        flight.flush();
-        ta_wait<0>();
-    } else if (warp == 6) {
+        flush();
+    } else if (warp == 8) {
         // ---------------- products (one thread)
         if (lane == 0) {
             constexpr uint32_t idesc_qk = umma_idesc(TA_BN);
             constexpr uint32_t idesc_pv = umma_idesc_b_mn(VB * 64);
-            const uint64_t q_desc = umma_desc_sw128(smem_addr(sQ));
-            const uint64_t k_desc = umma_desc_sw128(smem_addr(sK));
+            const uint64_t k_desc = umma_desc_sw128(smem_addr(smem));
             const uint64_t v_desc = umma_desc_mn_sw128(smem_addr(sV), TA_BAND, 1024);
             bool ok = true;
-            uint32_t slot = 0, use = 0;
+            int k_slot = 0, k_use = 0;
             auto give_up = [&]() {
                 if (!*abort_word && flag) atomicOr(flag, KB_FLAG_TIMEOUT);
                 *abort_word = 1;
                 ok = false;
             };
             auto issue_qk = [&](int n) {
-                for (int b = 0; b < key_bands; ++b) {
-                    if (!mbar_wait(k_full + slot, use & 1, abort_word)) {
-                        give_up();
-                        return;
-                    }
-                    tc_fence_after();
-                    const uint64_t qb = q_desc + (uint64_t)((b * TA_BAND) >> 4);
-                    const uint64_t kb = k_desc + (uint64_t)((slot * TA_BAND) >> 4);
-#pragma unroll
-                    for (int k = 0; k < 4; ++k)  // 16 columns = 32 bytes along the swizzled row
-                        umma_bf16(tmem_base + TA_S_COL + (n & 1) * TA_BN, qb + (uint64_t)(k * 2), kb + (uint64_t)(k * 2), idesc_qk, (b > 0 || k > 0) ? 1u : 0u);
-                    umma_commit(k_empty + slot);
-                    if (++slot == (uint32_t)stages) {
-                        slot = 0;
-                        ++use;
-                    }
+                if (!mbar_wait(k_full + k_slot, k_use & 1, abort_word)) {
+                    give_up();
+                    return;
                 }
+                tc_fence_after();
+                const uint64_t kb = k_desc + (uint64_t)((k_slot * k_bytes) >> 4);
+                const uint32_t s_at = tmem_base + S_COL + (n & 1) * TA_BN, q_at = tmem_base + Q_COL;
+#pragma unroll
+                for (int b = 0; b < TA_MAX_BANDS; ++b)
+                    if (b < key_bands) {
+#pragma unroll
+                        for (int k = 0; k < 4; ++k)  // 16 columns: 8 columns of the queries in tensor memory, 32 bytes along the keys' swizzled row
+                            umma_bf16_a_tmem(s_at, q_at + b * 32 + k * 8, kb + (uint64_t)((b * TA_BAND + k * 32) >> 4), idesc_qk, (b > 0 || k > 0) ? 1u : 0u);
+                    }
+                umma_commit(k_empty + k_slot);
                 umma_commit(s_full + (n & 1));
+                if (++k_slot == TA_K_STAGES) {
+                    k_slot = 0;
+                    ++k_use;
+                }
             };
-            if (!mbar_wait(q_full, 0, abort_word)) give_up();
+            if (!mbar_wait(q_stored, 0, abort_word)) give_up();
+            tc_fence_after();
             if (ok) issue_qk(0);
             if (ok && num_kt > 1) issue_qk(1);
             for (int n = 0; n < num_kt && ok; ++n) {
-                if (!mbar_wait(p_full + (n & 1), (n >> 1) & 1, abort_word) || !mbar_wait(v_full, n & 1, abort_word)) {
+                const int v_slot = n % TA_V_STAGES;
+                if (!mbar_wait(p_full + (n & 1), (n >> 1) & 1, abort_word) || !mbar_wait(v_full + v_slot, (n / TA_V_STAGES) & 1, abort_word)) {
                     give_up();
                     break;
                 }
                 tc_fence_after();
+                const uint64_t vb = v_desc + (uint64_t)((v_slot * v_bytes) >> 4);
 #pragma unroll
                 for (int ks = 0; ks < TA_BN / 16; ++ks)  // 16 keys: 8 columns of P in tensor memory, 16 rows (2 KB) of V
-                    umma_bf16_a_tmem(tmem_base + TA_O_COL, tmem_base + TA_S_COL + (n & 1) * TA_BN + ks * 8, v_desc + (uint64_t)(ks * 128), idesc_pv,
+                    umma_bf16_a_tmem(tmem_base + O_COL, tmem_base + S_COL + (n & 1) * TA_BN + ks * 8, vb + (uint64_t)(ks * 128), idesc_pv,
                                      (n > 0 || ks > 0) ? 1u : 0u);
-                umma_commit(v_empty);
+                umma_commit(v_empty + v_slot);
                 umma_commit(pv_done + (n & 1));
                 // the softmax holds S_n in registers (it has written P_n), and the pipe keeps the order of products: S_n's
                 // buffer takes tile n + 2
@@ -316,14 +325,35 @@ talking_attention_tc5_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, 
         float m_ref = -INFINITY;  // the maximum the row's P and O are scaled by
         float l = 0.0f;
         bool ok = true;
-        for (int n = 0; n < num_kt; ++n) {
+        // the row's queries, a band of 64 columns (32 of tensor memory) at a time
+        if (!mbar_wait(q_loaded, 0, abort_word)) ok = false;
+        if (ok) {
+            for (int b = 0; b < key_bands; ++b) {
+                const unsigned char* src = smem + k_bytes + (r * key_bands + b) * 128;
+                uint32_t band[32];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    const uint4 v = *reinterpret_cast<const uint4*>(src + ((i ^ (r & 7)) * 16));
+                    band[4 * i] = v.x;
+                    band[4 * i + 1] = v.y;
+                    band[4 * i + 2] = v.z;
+                    band[4 * i + 3] = v.w;
+                }
+                tmem_store32(lane_base + Q_COL + b * 32, band);
+            }
+            tmem_wait_st();
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(q_stored);
+        }
+        for (int n = 0; n < num_kt && ok; ++n) {
             const int key0 = key_of(n);
             if (!mbar_wait(s_full + (n & 1), (n >> 1) & 1, abort_word)) { ok = false; break; }
             tc_fence_after();
-            const uint32_t s_at = lane_base + TA_S_COL + (n & 1) * TA_BN;
-            uint32_t raw[4][32];
+            const uint32_t s_at = lane_base + S_COL + (n & 1) * TA_BN;
+            uint32_t raw[2][32];
 #pragma unroll
-            for (int c = 0; c < 4; ++c) tmem_load32_nowait(s_at + c * 32, raw[c]);
+            for (int c = 0; c < 2; ++c) tmem_load32_nowait(s_at + c * 32, raw[c]);
             tmem_wait_ld();
             // on the raw scores for a positive scale: the maximum is taken before the scale, which then enters the exponent's
             // argument with the reference as one fused multiply-add; a scale of another sign is applied first
@@ -361,32 +391,28 @@ talking_attention_tc5_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, 
 #pragma unroll
                 for (int c = 0; c < VB * 2; ++c) {
                     uint32_t o[32];
-                    tmem_load32_nowait(lane_base + TA_O_COL + c * 32, o);
+                    tmem_load32_nowait(lane_base + O_COL + c * 32, o);
                     tmem_wait_ld();
 #pragma unroll
                     for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
-                    tmem_store32(lane_base + TA_O_COL + c * 32, o);
+                    tmem_store32(lane_base + O_COL + c * 32, o);
                 }
                 tmem_wait_st();
                 l *= alpha;
             }
             const float base = m_ref == -INFINITY ? 0.0f : -m_ref;
             float sum4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+            uint32_t packed[32];
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                uint32_t packed[32];
-#pragma unroll
-                for (int c = 0; c < 64; c += 2) {
-                    const int at = half * 64 + c;
-                    const float s0 = __uint_as_float(raw[at >> 5][at & 31]), s1 = __uint_as_float(raw[at >> 5][(at & 31) + 1]);
-                    const float p0 = ta_ex2(fmaf(s0, sl2, base)), p1 = ta_ex2(fmaf(s1, sl2, base));
-                    sum4[c & 2] += p0;
-                    sum4[(c & 2) + 1] += p1;
-                    __nv_bfloat162 pair = __floats2bfloat162_rn(p0, p1);
-                    packed[c >> 1] = *reinterpret_cast<uint32_t*>(&pair);
-                }
-                tmem_store32(s_at + half * 32, packed);
+            for (int c = 0; c < TA_BN; c += 2) {
+                const float s0 = __uint_as_float(raw[c >> 5][c & 31]), s1 = __uint_as_float(raw[c >> 5][(c & 31) + 1]);
+                const float p0 = ta_ex2(fmaf(s0, sl2, base)), p1 = ta_ex2(fmaf(s1, sl2, base));
+                sum4[c & 2] += p0;
+                sum4[(c & 2) + 1] += p1;
+                __nv_bfloat162 pair = __floats2bfloat162_rn(p0, p1);
+                packed[c >> 1] = *reinterpret_cast<uint32_t*>(&pair);
             }
+            tmem_store32(s_at, packed);
             l += (sum4[0] + sum4[1]) + (sum4[2] + sum4[3]);
             tmem_wait_st();
             tc_fence_before();
@@ -402,7 +428,7 @@ talking_attention_tc5_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, 
 #pragma unroll
             for (int c = 0; c < VB * 2; ++c) {
                 uint32_t o[32];
-                tmem_load32_nowait(lane_base + TA_O_COL + c * 32, o);
+                tmem_load32_nowait(lane_base + O_COL + c * 32, o);
                 tmem_wait_ld();
                 if (valid) {
 #pragma unroll
@@ -426,25 +452,20 @@ talking_attention_tc5_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, 
     }
     tc_fence_before();
     __syncthreads();
-    if (warp == 6) {
+    if (warp == 8) {
         tc_fence_after();
         tmem_dealloc(tmem_base, TA_TMEM_COLUMNS);
     }
 }
 
-#define TA_SMEM_LIMIT (227 * 1024)
-#define TA_BAR_BYTES ((1 + 2 * TA_MAX_STAGES + 8) * 8 + 16)
+#define TA_SMEM_MAX ((TA_K_STAGES * TA_MAX_BANDS + TA_V_STAGES * 2) * TA_BAND + (2 * TA_K_STAGES + 2 * TA_V_STAGES + 8) * 8 + 16)
 
 static int ta_key_bands(int G, int D) { return (G * D + 63) / 64; }
 static int ta_value_bands(int D) { return (D + 63) / 64; }
-static int ta_stages(int G, int D) {
-    const int room = TA_SMEM_LIMIT - TA_BAR_BYTES - (ta_key_bands(G, D) + ta_value_bands(D)) * TA_BAND;
-    const int stages = room / TA_BAND;
-    return stages > TA_MAX_STAGES ? TA_MAX_STAGES : stages;
-}
 
 KB_EXPORT int kb_talking_attention_tc5_supported(int H, int G, int D) {
-    return G >= 1 && H >= 1 && H % G == 0 && H / G <= TA_BM && D >= 8 && D <= 128 && D % 8 == 0 && ta_stages(G, D) >= 2;
+    return G >= 1 && H >= 1 && H % G == 0 && H / G <= TA_BM && D >= 8 && D <= 128 && D % 8 == 0
+           && ta_key_bands(G, D) <= TA_MAX_BANDS;
 }
 
 // list_rows / list_starts: the request row and the first query of each tile of 128 / (H / G) queries of the step's portions.
@@ -458,8 +479,8 @@ KB_EXPORT int kb_talking_attention_tc5(const void* q, int q_stride, void* out, i
     if (count > 65535 || page_size < 1 || keep_first < 0 || q_stride % 8 || out_stride % 8
         || (((uintptr_t)q | (uintptr_t)out | (uintptr_t)k_cache | (uintptr_t)v_cache) % 16)) return KB_ERR_BAD_ARG;
     if ((long long)num_pages * page_size > 0x7fffffffLL) return KB_ERR_UNSUPPORTED_SIZE;
-    const int bands = ta_key_bands(G, D), vb = ta_value_bands(D), stages = ta_stages(G, D);
-    const size_t smem = (size_t)(bands + stages + vb) * TA_BAND + TA_BAR_BYTES;
+    const int bands = ta_key_bands(G, D), vb = ta_value_bands(D);
+    const size_t smem = TA_SMEM_MAX - (size_t)((TA_MAX_BANDS - bands) * TA_K_STAGES + (2 - vb) * TA_V_STAGES) * TA_BAND;
     int shift = -1;
     if ((page_size & (page_size - 1)) == 0) {
         shift = 0;
@@ -469,12 +490,12 @@ KB_EXPORT int kb_talking_attention_tc5(const void* q, int q_stride, void* out, i
     do {                                                                                                                                    \
         static bool configured = false;                                                                                                     \
         if (!configured) {                                                                                                                  \
-            cudaFuncSetAttribute(talking_attention_tc5_kernel<VB>, cudaFuncAttributeMaxDynamicSharedMemorySize, TA_SMEM_LIMIT);               \
+            cudaFuncSetAttribute(talking_attention_tc5_kernel<VB>, cudaFuncAttributeMaxDynamicSharedMemorySize, TA_SMEM_MAX);               \
             configured = true;                                                                                                              \
         }                                                                                                                                   \
         kb_launch(talking_attention_tc5_kernel<VB>, dim3(G, count), dim3(TA_THREADS), smem, stream, (const __nv_bfloat16*)q, q_stride,       \
                   (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, qo_indptr, seq_lens,        \
-                  block_table, max_pages, list_rows, list_starts, H, G, D, bands, stages, page_size, shift, num_pages, scale, window,        \
+                  block_table, max_pages, list_rows, list_starts, H, G, D, bands, page_size, shift, num_pages, scale, window,        \
                   keep_first, flag);                                                                                                        \
     } while (0)
     if (vb == 1) LAUNCH(1); else LAUNCH(2);

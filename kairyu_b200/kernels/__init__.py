@@ -667,19 +667,11 @@ def talking_prepare(
 
 
 def talking_attention_supported(num_q_heads: int, num_kv_heads: int, head_dim: int) -> bool:
-    """Sizes that the tensor-core kernels of attention over one wide key row take (csrc/talking_attention_tc5.cu: ``supported``,
-    csrc/talking_attention_decode.cu: ``td_shape``): heads of a multiple of 16 up to 128 columns, key rows that fit beside their
-    rings of buffers in shared memory (up to about 640 columns), up to 16 query heads a key/value head and 64 in all."""
-    if num_kv_heads < 1 or num_q_heads % num_kv_heads or num_q_heads // num_kv_heads > 16 or num_q_heads > 64 or head_dim % 16 or not 16 <= head_dim <= 128:
-        return False
-    width = num_kv_heads * head_dim
-    band = 128 * 128
-    bands, value_bands = -(-width // 64), -(-head_dim // 64)
-    if (227 * 1024 - 216 - (bands + value_bands) * band) // band < 2:
-        return False
-    rows, stride = 16 * -(-num_q_heads // 16), width + 8
-    two_stages = (rows * stride + 2 * 64 * stride + rows * 40) * 2 + (2 * rows * 34 + 3 * rows) * 4
-    return width <= 1024 and two_stages <= 220 * 1024
+    """Sizes that the tensor-core kernels of attention over one wide key row take (csrc/talking_attention_tc5.cu and
+    csrc/talking_attention_decode.cu: ``supported``): heads of a multiple of 16 up to 128 columns, key rows of up to 512, up to 16
+    query heads a key/value head and 32 in all."""
+    return (num_kv_heads >= 1 and num_q_heads % num_kv_heads == 0 and num_q_heads // num_kv_heads <= 16 and num_q_heads <= 32
+            and head_dim % 16 == 0 and 16 <= head_dim <= 128 and num_kv_heads * head_dim <= 512)
 
 
 def talking_attention_tile(num_q_heads: int, num_kv_heads: int) -> int:
@@ -736,11 +728,11 @@ def talking_attention(
             part_ml = ctx.workspace.flat("talk.part_ml", splits * count * num_q_heads * 2, torch.float32)
         fn = _fn("talking_attention_decode", "kb_talking_decode",
                  [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                  c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p])
+                  c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p])
         _check(fn(queries.data_ptr(), queries.stride(0), out.data_ptr(), out.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), ctx.seq_lens.data_ptr(),
                   block_table.data_ptr(), block_table.shape[1], ctx.decode_rows.data_ptr(), ctx.decode_tokens.data_ptr(), int(count), num_q_heads,
                   num_kv_heads, head_dim, page_size, num_pages, float(scale), int(window), int(keep_first), splits, _ptr(part_o), _ptr(part_ml),
-                  _stream()), what, launches=2 if splits > 1 else 1)
+                  _ptr(flag), _stream()), what, launches=2 if splits > 1 else 1)
 
 
 DIFF_ATTENTION_TILE = 64  # queries a tile of the tensor-core kernel for prompt portions
