@@ -13,9 +13,8 @@
 // strides and the weights' alignment alone, never on the batch.
 #include "common.cuh"
 
-#define GR_THREADS 256      // of the scalar form
-#define GR_VEC_THREADS 512  // of the vector form, at most: a row's loads are then all in flight at once up to 2,048 columns
-#define GR_CHUNKS 4         // four-column groups a thread of the vector form keeps
+#define GR_THREADS 256
+#define GR_CHUNKS 4  // four-column groups a thread of the vector form keeps at most: rows of up to 4 * 4 * 256 columns
 
 __device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
 __device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
@@ -32,6 +31,11 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
     raw.y = *reinterpret_cast<const unsigned*>(&hi);
     *reinterpret_cast<uint2*>(p) = raw;
 }
+// a weight vector of either type
+__device__ __forceinline__ float weight1(const void* p, int bf16, int i) {
+    return bf16 ? to_float(((const __nv_bfloat16*)p)[i]) : ((const float*)p)[i];
+}
+__device__ __forceinline__ float4 weight4(const void* p, int bf16, int i) { return bf16 ? load4((const __nv_bfloat16*)p + i) : load4((const float*)p + i); }
 __device__ __forceinline__ float gate_of(float g, float b) { return 1.0f / (1.0f + expf(-(g + b))); }
 
 struct GatedSum {
@@ -43,9 +47,11 @@ struct GatedSum {
     const void* extra;        // TA
     const void* gate;         // TA
     int gate_stride;
-    const void* bias;         // TB
+    const void* bias;
+    int bias_bf16;
     float mult;
-    const void* w;            // TW
+    const void* w;
+    int w_bf16;
     float eps;
     const float* origin;
     void* out;                // TA
@@ -54,8 +60,8 @@ struct GatedSum {
     int H;
 };
 
-// TY: the values' dtype, TA: the activations' (gate, extra, out), TB: gate bias, TW: norm weight
-template <typename TY, typename TA, typename TB, typename TW>
+// TY: the values' dtype, TA: the activations' (gate, extra, out)
+template <typename TY, typename TA>
 __global__ void __launch_bounds__(GR_THREADS) gated_residual_norm_kernel(const GatedSum p) {
     extern __shared__ float row[];
     __shared__ float scratch[32];
@@ -66,7 +72,7 @@ __global__ void __launch_bounds__(GR_THREADS) gated_residual_norm_kernel(const G
     const TY* values = (const TY*)p.values;
     const TA* gate = (const TA*)p.gate;
     const TA* extra = (const TA*)p.extra;
-    const TB* bias = (const TB*)p.bias;
+    const void* bias = p.bias;
     TA* out = (TA*)p.out + (size_t)r * p.out_stride;
     float* xr = p.x + (size_t)t * p.H;
     float ss = 0.0f;
@@ -84,64 +90,86 @@ __global__ void __launch_bounds__(GR_THREADS) gated_residual_norm_kernel(const G
             } else {
                 y = to_float(values[(size_t)t * p.H + i]);
             }
-            v += p.mult * gate_of(to_float(gate[(size_t)t * p.gate_stride + i]), bias ? to_float(bias[i]) : 0.0f) * y;
+            v += p.mult * gate_of(to_float(gate[(size_t)t * p.gate_stride + i]), bias ? weight1(bias, p.bias_bf16, i) : 0.0f) * y;
             if (!p.rows) xr[i] = v;
         }
         row[i] = v;
         ss += v * v;
     }
-    const TW* w = (const TW*)p.w;
+    const void* w = p.w;
     const float inv = w ? rsqrtf(block_sum(ss, scratch) / (float)p.H + p.eps) : 1.0f;
     for (int i = threadIdx.x; i < p.H; i += GR_THREADS) {
-        out[i] = from_float<TA>(w ? row[i] * inv * to_float(w[i]) : row[i]);
+        out[i] = from_float<TA>(w ? row[i] * inv * weight1(w, p.w_bf16, i) : row[i]);
         if (p.origin) out[p.H + i] = from_float<TA>(p.origin[(size_t)t * p.H + i]);
     }
 }
 
-template <typename TY, typename TA, typename TB, typename TW>
-__global__ void __launch_bounds__(GR_VEC_THREADS) gated_residual_norm_vec_kernel(const GatedSum p) {
+// CHUNKS: four-column groups a thread keeps
+template <typename TY, typename TA, int CHUNKS>
+__global__ void __launch_bounds__(GR_THREADS) gated_residual_norm_vec_kernel(const GatedSum p) {
     __shared__ float scratch[32];
     pdl_trigger();
     const int r = blockIdx.x;
     const int t = p.rows ? p.rows[r] : r;
     const int H = p.H;
-    const TB* bias = (const TB*)p.bias;
-    const TW* w = (const TW*)p.w;
+    const void* bias = p.bias;
+    const void* w = p.w;
     pdl_wait();
     const TY* values = (const TY*)p.values;
     TA* out = (TA*)p.out + (size_t)r * p.out_stride;
     float* xr = p.x + (size_t)t * H;
-    float4 kept[GR_CHUNKS];
+    // every load of the row goes out before the first store, so that they are all in flight together
+    float4 kept[CHUNKS], y[CHUNKS], g[CHUNKS];
+#pragma unroll
+    for (int c = 0; c < CHUNKS; ++c) {
+        const int i = (c * GR_THREADS + threadIdx.x) * 4;
+        if (i >= H) continue;
+        kept[c] = load4(xr + i);
+        if (values) {
+            g[c] = load4((const TA*)p.gate + (size_t)t * p.gate_stride + i);
+            if (!p.mix) y[c] = load4(values + (size_t)t * H + i);
+        }
+    }
+    if (p.mix) {
+#pragma unroll
+        for (int c = 0; c < CHUNKS; ++c) y[c] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        for (int k0 = 0; k0 < p.K; k0 += 2) {  // two of the token's rows at a time, in the order of k
+            const size_t pair = (size_t)t * p.K + k0;
+            const bool second = k0 + 1 < p.K;
+            const float m0 = p.mix[pair], m1 = second ? p.mix[pair + 1] : 0.0f;
+            const TY* row0 = values + (p.at ? (size_t)p.at[pair] : pair) * H;
+            const TY* row1 = second ? values + (p.at ? (size_t)p.at[pair + 1] : pair + 1) * H : row0;
+#pragma unroll
+            for (int c = 0; c < CHUNKS; ++c) {
+                const int i = (c * GR_THREADS + threadIdx.x) * 4;
+                if (i >= H) continue;
+                const float4 a = load4(row0 + i), b = load4(row1 + i);
+                y[c].x += m0 * a.x; y[c].y += m0 * a.y; y[c].z += m0 * a.z; y[c].w += m0 * a.w;
+                if (second) { y[c].x += m1 * b.x; y[c].y += m1 * b.y; y[c].z += m1 * b.z; y[c].w += m1 * b.w; }
+            }
+        }
+        if (p.extra) {
+#pragma unroll
+            for (int c = 0; c < CHUNKS; ++c) {
+                const int i = (c * GR_THREADS + threadIdx.x) * 4;
+                if (i >= H) continue;
+                const float4 e = load4((const TA*)p.extra + (size_t)t * H + i);
+                y[c].x += e.x; y[c].y += e.y; y[c].z += e.z; y[c].w += e.w;
+            }
+        }
+    }
     float ss = 0.0f;
 #pragma unroll
-    for (int c = 0; c < GR_CHUNKS; ++c) {
-        const int i = (c * (int)blockDim.x + threadIdx.x) * 4;
-        if (i >= H) break;
-        float4 v = load4(xr + i);
+    for (int c = 0; c < CHUNKS; ++c) {
+        const int i = (c * GR_THREADS + threadIdx.x) * 4;
+        if (i >= H) continue;
+        float4 v = kept[c];
         if (values) {
-            float4 y;
-            if (p.mix) {
-                y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-#pragma unroll 4
-                for (int k = 0; k < p.K; ++k) {
-                    const size_t pair = (size_t)t * p.K + k;
-                    const float m = p.mix[pair];
-                    const float4 part = load4(values + (p.at ? (size_t)p.at[pair] : pair) * H + i);
-                    y.x += m * part.x; y.y += m * part.y; y.z += m * part.z; y.w += m * part.w;
-                }
-                if (p.extra) {
-                    const float4 e = load4((const TA*)p.extra + (size_t)t * H + i);
-                    y.x += e.x; y.y += e.y; y.z += e.z; y.w += e.w;
-                }
-            } else {
-                y = load4(values + (size_t)t * H + i);
-            }
-            const float4 g = load4((const TA*)p.gate + (size_t)t * p.gate_stride + i);
-            const float4 b = bias ? load4(bias + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            v.x += p.mult * gate_of(g.x, b.x) * y.x;
-            v.y += p.mult * gate_of(g.y, b.y) * y.y;
-            v.z += p.mult * gate_of(g.z, b.z) * y.z;
-            v.w += p.mult * gate_of(g.w, b.w) * y.w;
+            const float4 b = bias ? weight4(bias, p.bias_bf16, i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            v.x += p.mult * gate_of(g[c].x, b.x) * y[c].x;
+            v.y += p.mult * gate_of(g[c].y, b.y) * y[c].y;
+            v.z += p.mult * gate_of(g[c].z, b.z) * y[c].z;
+            v.w += p.mult * gate_of(g[c].w, b.w) * y[c].w;
             if (!p.rows) store4(xr + i, v);
         }
         kept[c] = v;
@@ -149,12 +177,12 @@ __global__ void __launch_bounds__(GR_VEC_THREADS) gated_residual_norm_vec_kernel
     }
     const float inv = w ? rsqrtf(block_sum(ss, scratch) / (float)H + p.eps) : 1.0f;
 #pragma unroll
-    for (int c = 0; c < GR_CHUNKS; ++c) {
-        const int i = (c * (int)blockDim.x + threadIdx.x) * 4;
-        if (i >= H) break;
+    for (int c = 0; c < CHUNKS; ++c) {
+        const int i = (c * GR_THREADS + threadIdx.x) * 4;
+        if (i >= H) continue;
         float4 v = kept[c];
         if (w) {
-            const float4 n = load4(w + i);
+            const float4 n = weight4(w, p.w_bf16, i);
             v = make_float4(v.x * inv * n.x, v.y * inv * n.y, v.z * inv * n.z, v.w * inv * n.w);
         }
         store4(out + i, v);
@@ -163,21 +191,12 @@ __global__ void __launch_bounds__(GR_VEC_THREADS) gated_residual_norm_vec_kernel
 }
 
 template <typename TY, typename TA>
-static int launch_gated(const GatedSum& p, int R, int bias_bf16, int w_bf16, bool vec, cudaStream_t stream) {
-    const size_t smem = vec ? 0 : (size_t)p.H * sizeof(float);
-    const int wanted = (p.H / 4 + 31) / 32 * 32;
-    const int threads = wanted > GR_VEC_THREADS ? GR_VEC_THREADS : wanted;
-#define LAUNCH(TB, TW)                                                                                                          \
-    do {                                                                                                                        \
-        if (vec) kb_launch(gated_residual_norm_vec_kernel<TY, TA, TB, TW>, dim3(R), dim3(threads), smem, stream, p);              \
-        else kb_launch(gated_residual_norm_kernel<TY, TA, TB, TW>, dim3(R), dim3(GR_THREADS), smem, stream, p);                   \
-    } while (0)
-    if (bias_bf16) {
-        if (w_bf16) LAUNCH(__nv_bfloat16, __nv_bfloat16); else LAUNCH(__nv_bfloat16, float);
-    } else {
-        if (w_bf16) LAUNCH(float, __nv_bfloat16); else LAUNCH(float, float);
-    }
-#undef LAUNCH
+static int launch_gated(const GatedSum& p, int R, bool vec, cudaStream_t stream) {
+    const int chunks = (p.H + 4 * GR_THREADS - 1) / (4 * GR_THREADS);
+    if (!vec) kb_launch(gated_residual_norm_kernel<TY, TA>, dim3(R), dim3(GR_THREADS), (size_t)p.H * sizeof(float), stream, p);
+    else if (chunks == 1) kb_launch(gated_residual_norm_vec_kernel<TY, TA, 1>, dim3(R), dim3(GR_THREADS), 0, stream, p);
+    else if (chunks == 2) kb_launch(gated_residual_norm_vec_kernel<TY, TA, 2>, dim3(R), dim3(GR_THREADS), 0, stream, p);
+    else kb_launch(gated_residual_norm_vec_kernel<TY, TA, GR_CHUNKS>, dim3(R), dim3(GR_THREADS), 0, stream, p);
     return kb_launch_result();
 }
 
@@ -189,13 +208,13 @@ KB_EXPORT int kb_gated_residual_norm(float* x, const void* values, int values_bf
     if (!x || !out || (values && !gate)) return KB_ERR_NULL;
     if (H < 1 || H > 12000 || K < 1) return KB_ERR_UNSUPPORTED_SIZE;  // the scalar form keeps the row in 48 KB of shared memory
     if (out_stride < (origin ? 2 * H : H)) return KB_ERR_BAD_ARG;
-    const GatedSum p = {x, values, mix, at, K, extra, gate, gate_stride, bias, mult, w, eps, origin, out, out_stride, rows, H};
+    const GatedSum p = {x, values, mix, at, K, extra, gate, gate_stride, bias, bias_bf16, mult, w, w_bf16, eps, origin, out, out_stride, rows, H};
     const uintptr_t all = (uintptr_t)x | (uintptr_t)values | (uintptr_t)extra | (uintptr_t)gate | (uintptr_t)bias | (uintptr_t)w | (uintptr_t)origin | (uintptr_t)out;
-    const bool vec = H % 4 == 0 && H <= 4 * GR_CHUNKS * GR_VEC_THREADS && gate_stride % 4 == 0 && out_stride % 4 == 0 && all % 16 == 0;
+    const bool vec = H % 4 == 0 && H <= 4 * GR_CHUNKS * GR_THREADS && gate_stride % 4 == 0 && out_stride % 4 == 0 && all % 16 == 0;
     if (act_bf16) {
-        if (values_bf16) return launch_gated<__nv_bfloat16, __nv_bfloat16>(p, R, bias_bf16, w_bf16, vec, stream);
-        return launch_gated<float, __nv_bfloat16>(p, R, bias_bf16, w_bf16, vec, stream);
+        if (values_bf16) return launch_gated<__nv_bfloat16, __nv_bfloat16>(p, R, vec, stream);
+        return launch_gated<float, __nv_bfloat16>(p, R, vec, stream);
     }
     if (values_bf16) return KB_ERR_BAD_ARG;
-    return launch_gated<float, float>(p, R, bias_bf16, w_bf16, vec, stream);
+    return launch_gated<float, float>(p, R, vec, stream);
 }

@@ -720,19 +720,37 @@ def talking_attention(
     count = ctx.num_decode_rows
     if count:
         keys = ctx.max_seq_len if window <= 0 else min(ctx.max_seq_len, window + keep_first)
-        splits_fn = _fn("talking_attention_decode", "kb_talking_decode_splits", [c_int] * 5)
-        splits = int(splits_fn(count, int(keys), num_q_heads, num_kv_heads, head_dim))
+        splits_fn = _fn("talking_attention_decode", "kb_talking_decode_splits", [c_int] * 6)
+        splits = int(splits_fn(count, int(keys), num_q_heads, num_kv_heads, head_dim, page_size))
         part_o = part_ml = None
         if splits > 1:
             part_o = ctx.workspace.flat("talk.part_o", splits * count * num_q_heads * head_dim, torch.float32)
             part_ml = ctx.workspace.flat("talk.part_ml", splits * count * num_q_heads * 2, torch.float32)
+        maps = (None, None)
+        if _fn("talking_attention_decode", "kb_talking_decode_uses_tma", [c_int] * 4)(num_q_heads, num_kv_heads, head_dim, page_size):
+            maps = (_wide_row_map(k_cache), _wide_row_map(v_cache))
         fn = _fn("talking_attention_decode", "kb_talking_decode",
-                 [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                 [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                   c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p])
-        _check(fn(queries.data_ptr(), queries.stride(0), out.data_ptr(), out.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), ctx.seq_lens.data_ptr(),
+        _check(fn(*maps, queries.data_ptr(), queries.stride(0), out.data_ptr(), out.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), ctx.seq_lens.data_ptr(),
                   block_table.data_ptr(), block_table.shape[1], ctx.decode_rows.data_ptr(), ctx.decode_tokens.data_ptr(), int(count), num_q_heads,
                   num_kv_heads, head_dim, page_size, num_pages, float(scale), int(window), int(keep_first), splits, _ptr(part_o), _ptr(part_ml),
                   _ptr(flag), _stream()), what, launches=2 if splits > 1 else 1)
+
+
+def _wide_row_map(cache: torch.Tensor) -> int:
+    """Host address of a cached TMA descriptor of one layer's key (or value) pages as rows of all heads side by side."""
+    key = ("wide rows", cache.data_ptr(), tuple(cache.shape))
+    held = _held_map(key)
+    if held is None:
+        held = ctypes.create_string_buffer(128 + 64)
+        address = (ctypes.addressof(held) + 63) & ~63
+        fn = _fn("talking_attention_decode", "kb_talking_decode_encode_map", [c_void_p, c_void_p, ctypes.c_longlong, c_int, c_int])
+        code = fn(address, cache.data_ptr(), cache.shape[0], cache.shape[1], cache.shape[2] * cache.shape[3])
+        if code != 0:
+            raise KernelError(f"tensor map encoding of the cache's rows failed with code {code}")
+        _keep_map(key, held)
+    return (ctypes.addressof(held) + 63) & ~63
 
 
 DIFF_ATTENTION_TILE = 64  # queries a tile of the tensor-core kernel for prompt portions
