@@ -66,7 +66,7 @@ def diff_attention_generic(q, out, k_cache, v_cache, *, positions, row_ids, bloc
             out[t, h * vdim : (h + 1) * vdim] = o.to(out.dtype)
 
 
-def moe_route_scores(logits, correction, top, ids, weights, *, groups=1, keep=1, scale=1.0, score="softmax"):
+def moe_route_scores(logits, correction, top, ids, weights, *, groups=1, keep=1, scale=1.0, score="softmax", renormalise=False):
     outputs = logits.shape[1]
     per = outputs // groups
     for t in range(logits.shape[0]):
@@ -78,10 +78,10 @@ def moe_route_scores(logits, correction, top, ids, weights, *, groups=1, keep=1,
         allowed = [e for e in range(outputs) if e // per in kept]
         chosen = sorted(allowed, key=lambda e: (-float(c[e]), e))[:top]
         ids[t] = torch.tensor(chosen, dtype=torch.int32)
-        weights[t] = s[chosen] * scale
+        weights[t] = s[chosen] / (s[chosen].sum() + 1e-20) * scale if renormalise else s[chosen] * scale
 
 
-def moe_grouped(a, weight, out, plan, *, top, gated, limit=0.0, alpha=1.702, shift=1.0):
+def moe_grouped(a, weight, out, plan, *, top, gated, activation=None, limit=0.0, alpha=1.702, shift=1.0):
     for place, pair in enumerate(plan["sorted"]):
         expert = plan["experts"][pair]
         if expert >= weight.shape[0]:
@@ -93,6 +93,8 @@ def moe_grouped(a, weight, out, plan, *, top, gated, limit=0.0, alpha=1.702, shi
             g = both[:half].clamp(max=limit)
             u = both[half:].clamp(min=-limit, max=limit)
             out[place] = (g * torch.sigmoid(alpha * g) * (u + shift)).to(out.dtype)
+        elif activation is not None:
+            out[place] = (torch.relu(w @ a[pair // top].float()) ** 2).to(out.dtype)
         else:
             out[pair] = w @ a[place].float()
 

@@ -37,6 +37,12 @@ def visible(n, size, keep_first):
     return (j <= i) & ((i - j < size) | (j < keep_first))
 
 
+def window_of(m, n):
+    """(size, kept first tokens) of a mixer's mask; without one every key stays in sight."""
+    mask = m.get("mask")
+    return (mask["size"], mask.get("keep_first", 0)) if mask else (n, 0)
+
+
 def mix_heads(scores, talk):
     """scores [heads, n, n] -> sum over g of talk[h, g] * scores[g]."""
     return torch.einsum("hg,gij->hij", talk, scores)
@@ -53,7 +59,7 @@ def attention(h, w, m):
     own = [head // (H // G) for head in range(H)]
     scores = torch.stack([q[:, head] @ k[:, own[head]].T for head in range(H)]) * m["scale"]
     scores = mix_heads(scores, w["talk"])
-    scores = scores.masked_fill(~visible(n, m["mask"]["size"], m["mask"]["keep_first"]), -math.inf)
+    scores = scores.masked_fill(~visible(n, *window_of(m, n)), -math.inf)
     p = torch.softmax(scores, dim=-1)
     mixed = torch.cat([p[head] @ values[:, own[head]] for head in range(H)], dim=-1)
     return mixed @ w["o"].T
