@@ -32,8 +32,8 @@ and the rows left in sorted order; float32 and other sizes run this package's ow
 (gate and up with the activation in the epilogue, then down).  Nothing comes back to the host, so
 the work can sit in a captured graph.  Either way there is one row per pair at the end;
 ``forward(..., combine=False)`` hands those, the router's weights and where each row lies on
-(``kernels.WeightedRows``) for a kernel that adds them on its way (with an ungated-by-a-number shared expert's rows beside
-them), otherwise they are added here.
+(``kernels.WeightedRows``) for a kernel that adds them on its way (beside them the rows of a shared expert
+without a gate of its own), otherwise they are added here.
 """
 
 from __future__ import annotations
