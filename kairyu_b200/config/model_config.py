@@ -30,6 +30,7 @@ class RopeScaling:
     beta_slow: float = 1.0
     mscale: float | None = None
     mscale_all_dim: float | None = None
+    amplitude: float | None = None  # yarn: the factor on cos and sin, where a design states it outright
 
 
 @dataclass(frozen=True)

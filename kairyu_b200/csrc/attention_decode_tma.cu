@@ -119,7 +119,7 @@ attention_decode_tma_body(const CUtensorMap& map_k, const CUtensorMap& map_v,
                           const int* __restrict__ decode_tokens, int Hq, int Hkv, int page_size, int page_shift,
                           int num_pages, float scale, int window, int num_splits, float* __restrict__ part_o,
                           float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out, int out_stride, int combine,
-                          const float* __restrict__ sinks, const __nv_bfloat16* __restrict__ gate, int gate_stride, int* flag) {
+                          const float* __restrict__ sinks, const __nv_bfloat16* __restrict__ gate, int gate_stride, const KbSoftcap& cap, int* flag) {
     using S = TmaSmem<D, ST>;
     constexpr int HALVES = S::HALVES;
     static_assert(!JOINED || HALVES == 1, "keys and values share a copy at head_dim 64 only");
@@ -294,8 +294,8 @@ attention_decode_tma_body(const CUtensorMap& map_k, const CUtensorMap& map_v,
                 for (int e = 0; e < 2; ++e) {
                     const int key = key_base + nt * 8 + e;
                     const bool ok = key < seq_len && key >= key_lo;
-                    s[nt][e] = ok ? s[nt][e] * sl2 : -INFINITY;
-                    s[nt][2 + e] = ok ? s[nt][2 + e] * sl2 : -INFINITY;
+                    s[nt][e] = ok ? softcap_score(s[nt][e], sl2, cap) : -INFINITY;
+                    s[nt][2 + e] = ok ? softcap_score(s[nt][2 + e], sl2, cap) : -INFINITY;
                 }
             }
             float mx0 = fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1]));
@@ -427,10 +427,10 @@ attention_decode_tma_body(const CUtensorMap& map_k, const CUtensorMap& map_v,
         const int* __restrict__ decode_rows, const int* __restrict__ decode_tokens, int Hq, int Hkv, int page_size,          \
         int page_shift, int num_pages, float scale, int window, int num_splits, float* __restrict__ part_o,                  \
         float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out, int out_stride, int combine,                         \
-        const float* __restrict__ sinks, const __nv_bfloat16* __restrict__ gate, int gate_stride, int* flag
+        const float* __restrict__ sinks, const __nv_bfloat16* __restrict__ gate, int gate_stride, const KbSoftcap cap, int* flag
 #define DECODE_TMA_ARGS                                                                                                     \
     map_k, map_v, q, q_stride, seq_lens, block_table, max_pages, decode_rows, decode_tokens, Hq, Hkv, page_size, page_shift, \
-        num_pages, scale, window, num_splits, part_o, part_ml, out, out_stride, combine, sinks, gate, gate_stride, flag
+        num_pages, scale, window, num_splits, part_o, part_ml, out, out_stride, combine, sinks, gate, gate_stride, cap, flag
 
 template <int D, bool JOINED, int ST>
 __global__ void __launch_bounds__(TMA_THREADS) attention_decode_tma_kernel(DECODE_TMA_PARAMS) {
@@ -558,8 +558,8 @@ template <int D, bool JOINED, int ST = TmaStages<D>::value>
 int launch(const CUtensorMap* mk, const CUtensorMap* mv, const __nv_bfloat16* q, int q_stride, const int* seq_lens,
            const int* block_table, int max_pages, const int* decode_rows, const int* decode_tokens, int num_rows, int Hq,
            int Hkv, int page_size, int num_pages, float scale, int window, int num_splits, float* part_o, float* part_ml,
-           __nv_bfloat16* out, int out_stride, int combine, const float* sinks, const __nv_bfloat16* gate, int gate_stride, int* flag,
-           cudaStream_t stream) {
+           __nv_bfloat16* out, int out_stride, int combine, const float* sinks, const __nv_bfloat16* gate, int gate_stride,
+           const KbSoftcap& cap, int* flag, cudaStream_t stream) {
     const size_t smem = TmaSmem<D, ST>::TOTAL;
     cudaError_t e = cudaFuncSetAttribute(attention_decode_tma_kernel<D, JOINED, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
@@ -568,7 +568,7 @@ int launch(const CUtensorMap* mk, const CUtensorMap* mv, const __nv_bfloat16* q,
     dim3 grid(num_rows, Hkv, num_splits);
     kb_launch(attention_decode_tma_kernel<D, JOINED, ST>, dim3(grid), dim3(TMA_THREADS), smem, stream, *mk, *mv, q, q_stride, seq_lens,
               block_table, max_pages, decode_rows, decode_tokens, Hq, Hkv, page_size, shift, num_pages, scale,
-              window, num_splits, part_o, part_ml, out, out_stride, combine, sinks, gate, gate_stride, flag);
+              window, num_splits, part_o, part_ml, out, out_stride, combine, sinks, gate, gate_stride, cap, flag);
     return kb_launch_result();
 }
 
@@ -678,11 +678,12 @@ KB_EXPORT int kb_attention_encode_joined_map(void* map_out, const void* base_k, 
 // and written with more than one split).  sinks (optional): one fp32 logit a query head whose exp joins the
 // softmax's denominator; gate (optional): bf16 [tokens, gate_stride] laid out as out, by whose sigmoid the result
 // is multiplied.  Both act where a row's result is divided: in the kernel with one split, in the merge kernel else.
+// softcap (optional): a host KbSoftcap (softcap.cuh).
 KB_EXPORT int kb_attention_decode_tma(const void* map_k, const void* map_v, const void* q, int q_stride, void* out, int out_stride,
                                       const int* seq_lens, const int* block_table, int max_pages, const int* decode_rows,
                                       const int* decode_tokens, int num_rows, int Hq, int Hkv, int D, int page_size, int num_pages,
                                       float scale, int window, int num_splits, float* part_o, float* part_ml, int joined,
-                                      const float* sinks, const void* gate, int gate_stride, int* flag, cudaStream_t stream) {
+                                      const float* sinks, const void* gate, int gate_stride, const void* softcap, int* flag, cudaStream_t stream) {
     if (num_rows == 0) return 0;
     if (joined && D != 64) return KB_ERR_UNSUPPORTED_SIZE;
     if (joined) map_v = map_k;
@@ -698,7 +699,7 @@ KB_EXPORT int kb_attention_decode_tma(const void* map_k, const void* map_v, cons
     int rc;
 #define ARGS mk, mv, (const __nv_bfloat16*)q, q_stride, seq_lens, block_table, max_pages, decode_rows, decode_tokens, num_rows, Hq, \
              Hkv, page_size, num_pages, scale, window, num_splits, part_o, part_ml, (__nv_bfloat16*)out, out_stride, combine, sinks,    \
-             (const __nv_bfloat16*)gate, gate_stride, flag, stream
+             (const __nv_bfloat16*)gate, gate_stride, kb_softcap_of(softcap), flag, stream
     switch (D) {
         case 64: {
             // a grid that four-stage blocks cannot hold at once runs with three stages, four blocks an SM

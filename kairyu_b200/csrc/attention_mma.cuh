@@ -15,6 +15,7 @@
 // (multiples of DEC_SPLIT), so a row's result depends only on its own length.
 #pragma once
 #include "common.cuh"
+#include "softcap.cuh"
 
 #define TILE_N 64
 #define MMA_THREADS 128
@@ -201,7 +202,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
                          int max_pages, const int* __restrict__ tile_rows,
                          const int* __restrict__ tile_starts, int Hq, int Hkv, int D, int page_size,
                          int num_pages, float scale, int window, const float* __restrict__ sinks,
-                         const __nv_bfloat16* __restrict__ gate, int gate_stride, int* flag) {
+                         const __nv_bfloat16* __restrict__ gate, int gate_stride, const KbSoftcap cap, int* flag) {
     pdl_wait();
     extern __shared__ __align__(16) unsigned char smem_raw[];
     constexpr int STRIDE = Tile<DP>::STRIDE;
@@ -344,8 +345,8 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
                         ok0 = key <= qpos0 && (window <= 0 || key > qpos0 - window);
                         ok1 = key <= qpos1 && (window <= 0 || key > qpos1 - window);
                     }
-                    s[mt][nt][e] = ok0 ? s[mt][nt][e] * sl2 : -INFINITY;
-                    s[mt][nt][2 + e] = ok1 ? s[mt][nt][2 + e] * sl2 : -INFINITY;
+                    s[mt][nt][e] = ok0 ? softcap_score(s[mt][nt][e], sl2, cap) : -INFINITY;
+                    s[mt][nt][2 + e] = ok1 ? softcap_score(s[mt][nt][2 + e], sl2, cap) : -INFINITY;
                     mx0 = fmaxf(mx0, s[mt][nt][e]);
                     mx1 = fmaxf(mx1, s[mt][nt][2 + e]);
                 }
@@ -483,7 +484,7 @@ attention_decode_split_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                               int max_pages, const int* __restrict__ decode_rows,
                               const int* __restrict__ decode_tokens, int Hq, int Hkv, int D,
                               int page_size, int num_pages, float scale, int window, int num_splits,
-                              float* __restrict__ part_o, float* __restrict__ part_ml, int* flag) {
+                              float* __restrict__ part_o, float* __restrict__ part_ml, const KbSoftcap cap, int* flag) {
     pdl_wait();
     extern __shared__ __align__(16) unsigned char smem_raw[];
     constexpr int STRIDE = Tile<DP>::STRIDE;
@@ -597,8 +598,8 @@ attention_decode_split_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
             for (int e = 0; e < 2; ++e) {
                 const int key = key_base + nt * 8 + e;
                 const bool ok = key < key_end && key >= key_lo_all;
-                s[nt][e] = ok ? s[nt][e] * sl2 : -INFINITY;
-                s[nt][2 + e] = ok ? s[nt][2 + e] * sl2 : -INFINITY;
+                s[nt][e] = ok ? softcap_score(s[nt][e], sl2, cap) : -INFINITY;
+                s[nt][2 + e] = ok ? softcap_score(s[nt][2 + e], sl2, cap) : -INFINITY;
             }
         }
         float mx0 = fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1]));
@@ -784,14 +785,14 @@ static int launch_prefill(const __nv_bfloat16* q, int q_stride, __nv_bfloat16* o
                           const int* qo_indptr, const int* seq_lens, const int* block_table,
                           int max_pages, const int* tile_rows, const int* tile_starts, int num_tiles,
                           int Hq, int Hkv, int D, int page_size, int num_pages, float scale,
-                          int window, const float* sinks, const __nv_bfloat16* gate, int gate_stride, int* flag, cudaStream_t stream) {
+                          int window, const float* sinks, const __nv_bfloat16* gate, int gate_stride, const KbSoftcap& cap, int* flag, cudaStream_t stream) {
     const size_t smem = prefill_smem<DP, MT>();
     cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<DP, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     dim3 grid(Hq, num_tiles);
     kb_launch(attention_prefill_kernel<DP, MT>, dim3(grid), dim3(MMA_THREADS), smem, stream, 
         q, q_stride, out, out_stride, k_cache, v_cache, qo_indptr, seq_lens, block_table, max_pages,
-        tile_rows, tile_starts, Hq, Hkv, D, page_size, num_pages, scale, window, sinks, gate, gate_stride, flag);
+        tile_rows, tile_starts, Hq, Hkv, D, page_size, num_pages, scale, window, sinks, gate, gate_stride, cap, flag);
     return kb_launch_result();
 }
 
@@ -800,14 +801,14 @@ static int launch_decode(const __nv_bfloat16* q, int q_stride, const __nv_bfloat
                          const __nv_bfloat16* v_cache, const int* seq_lens, const int* block_table,
                          int max_pages, const int* decode_rows, const int* decode_tokens, int num_rows,
                          int Hq, int Hkv, int D, int page_size, int num_pages, float scale, int window,
-                         int num_splits, float* part_o, float* part_ml, int* flag, cudaStream_t stream) {
+                         int num_splits, float* part_o, float* part_ml, const KbSoftcap& cap, int* flag, cudaStream_t stream) {
     const size_t smem = decode_smem<DP>();
     cudaError_t e = cudaFuncSetAttribute(attention_decode_split_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     dim3 grid(num_rows, Hkv, num_splits);
     kb_launch(attention_decode_split_kernel<DP>, dim3(grid), dim3(MMA_THREADS), smem, stream, 
         q, q_stride, k_cache, v_cache, seq_lens, block_table, max_pages, decode_rows, decode_tokens,
-        Hq, Hkv, D, page_size, num_pages, scale, window, num_splits, part_o, part_ml, flag);
+        Hq, Hkv, D, page_size, num_pages, scale, window, num_splits, part_o, part_ml, cap, flag);
     return kb_launch_result();
 }
 

@@ -48,6 +48,7 @@
 // other roles leave through a shared abort word, and the block frees its TMEM and returns.
 // Sizes: head_dim 64 or 128, page_size a power of two from 8 up; others go to the mma.sync
 // kernel of attention_mma.cuh.
+#include "softcap.cuh"
 #include "umma.cuh"
 
 #define FA_THREADS 192
@@ -92,10 +93,27 @@ __device__ __forceinline__ float2 fadd2(float2 a, float2 b) {
     asm("add.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(*reinterpret_cast<uint64_t*>(&a)), "l"(*reinterpret_cast<uint64_t*>(&b)));
     return *reinterpret_cast<float2*>(&d);
 }
+__device__ __forceinline__ float2 fmul2(float2 a, float2 b) {
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(*reinterpret_cast<uint64_t*>(&a)), "l"(*reinterpret_cast<uint64_t*>(&b)));
+    return *reinterpret_cast<float2*>(&d);
+}
 __device__ __forceinline__ float max3(float a, float b, float c) {
     float d;
     asm("max.f32 %0, %1, %2, %3;\n" : "=f"(d) : "f"(a), "f"(b), "f"(c));
     return d;
+}
+
+// Two raw scores -> two capped scores in base 2 (softcap.cuh); both forms of the cap are uniform over the launch.
+__device__ __forceinline__ float2 fa_softcap_near(float2 x, const KbSoftcap& cap) {
+    const float2 z = fmul2(x, x);
+    float2 p = ffma2(z, make_float2(cap.c[3], cap.c[3]), make_float2(cap.c[2], cap.c[2]));
+    p = ffma2(z, p, make_float2(cap.c[1], cap.c[1]));
+    p = ffma2(z, p, make_float2(cap.c[0], cap.c[0]));
+    return fmul2(x, p);
+}
+__device__ __forceinline__ float fa_softcap_full(float x, const KbSoftcap& cap) {
+    return fmaf(-2.0f * cap.b, __fdividef(1.0f, 1.0f + ex2_ftz(cap.a * x)), cap.b);
 }
 
 template <int D>
@@ -116,7 +134,7 @@ struct FaCfg {
     static constexpr int BLOCKS_PER_SM = 2;
 };
 
-template <int D>
+template <int D, bool CAP>
 __global__ void __launch_bounds__(FA_THREADS, FaCfg<D>::BLOCKS_PER_SM)
 attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                              const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out, int out_stride,
@@ -125,7 +143,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
                              const int* __restrict__ tile_starts, int num_tiles, int Hq, int Hkv, int page_size, int page_shift,
                              int num_pages, float scale, int window, int merged, int paired, int splits, float* __restrict__ part_o,
                              float* __restrict__ part_ml, const float* __restrict__ sinks, const __nv_bfloat16* __restrict__ gate,
-                             int gate_stride, int* flag) {
+                             int gate_stride, const KbSoftcap cap, int* flag) {
     using Cfg = FaCfg<D>;
     constexpr int BANDS = Cfg::BANDS;
     extern __shared__ __align__(1024) unsigned char smem[];
@@ -383,7 +401,7 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
         const int r = quarter * 32 + lane;
         const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16);
         const int soft_tid = threadIdx.x - 64;  // 0..127
-        const float sl2 = scale * FA_LOG2E;
+        const float sl2 = CAP ? 1.0f : scale * FA_LOG2E;  // capped scores come with the scale in them
         bool ok = true;
         int g0 = 0;
         for (int part = 0; part < num_parts && ok; ++part) {
@@ -418,6 +436,19 @@ attention_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
                 float tt[FA_BN];
 #pragma unroll
                 for (int c = 0; c < FA_BN; ++c) tt[c] = __uint_as_float(raw[c >> 5][c & 31]);
+                if constexpr (CAP) {
+                    if (cap.mode == KB_SOFTCAP_NEAR) {
+#pragma unroll
+                        for (int c = 0; c < FA_BN; c += 2) {
+                            const float2 y = fa_softcap_near(make_float2(tt[c], tt[c + 1]), cap);
+                            tt[c] = y.x;
+                            tt[c + 1] = y.y;
+                        }
+                    } else {
+#pragma unroll
+                        for (int c = 0; c < FA_BN; ++c) tt[c] = fa_softcap_full(tt[c], cap);
+                    }
+                }
                 if (key0 + FA_BN - 1 > first_pos || key0 < lo_last) {  // the diagonal or the window's edge crosses this tile
 #pragma unroll
                     for (int c = 0; c < FA_BN; ++c) {
@@ -611,6 +642,7 @@ struct FbCfg {  // head_dim 128
 };
 
 // tile_rows / tile_starts list tiles of 256 queries here.
+template <bool CAP>
 __global__ void __launch_bounds__(FB_THREADS, 1)
 attention_prefill_tc5_two_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                                  const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out, int out_stride,
@@ -618,7 +650,7 @@ attention_prefill_tc5_two_kernel(const __grid_constant__ CUtensorMap map_q, cons
                                  const int* __restrict__ block_table, int max_pages, const int* __restrict__ tile_rows,
                                  const int* __restrict__ tile_starts, int num_tiles, int Hq, int Hkv, int page_size, int page_shift,
                                  int num_pages, float scale, int window, int merged, const float* __restrict__ sinks,
-                                 const __nv_bfloat16* __restrict__ gate, int gate_stride, int* flag) {
+                                 const __nv_bfloat16* __restrict__ gate, int gate_stride, const KbSoftcap cap, int* flag) {
     using Cfg = FbCfg;
     constexpr int D = Cfg::D;
     constexpr int BANDS = Cfg::BANDS;
@@ -858,7 +890,7 @@ attention_prefill_tc5_two_kernel(const __grid_constant__ CUtensorMap map_q, cons
         const uint32_t s_col = lane_base + Cfg::S_COL + x * FB_BN;
         const uint32_t o_col = lane_base + Cfg::O_COL + x * D;
         const int soft_tid = (warp - 4 - 4 * x) * 32 + lane;  // 0..127 within the group
-        const float sl2 = scale * FA_LOG2E;
+        const float sl2 = CAP ? 1.0f : scale * FA_LOG2E;  // capped scores come with the scale in them
         bool ok = true;
         const Side mine = x ? side_b : side_a;
         if (mine.rows > 0) {
@@ -880,6 +912,19 @@ attention_prefill_tc5_two_kernel(const __grid_constant__ CUtensorMap map_q, cons
 #pragma unroll
                 for (int part = 0; part < FB_BN / 32; ++part) tmem_load32_nowait(s_col + part * 32, raw[part]);
                 tmem_wait_ld();
+                if constexpr (CAP) {
+                    if (cap.mode == KB_SOFTCAP_NEAR) {
+#pragma unroll
+                        for (int c = 0; c < FB_BN; c += 2) {
+                            const float2 y = fa_softcap_near(make_float2(__uint_as_float(raw[c >> 5][c & 31]), __uint_as_float(raw[c >> 5][(c & 31) + 1])), cap);
+                            raw[c >> 5][c & 31] = __float_as_uint(y.x);
+                            raw[c >> 5][(c & 31) + 1] = __float_as_uint(y.y);
+                        }
+                    } else {
+#pragma unroll
+                        for (int c = 0; c < FB_BN; ++c) raw[c >> 5][c & 31] = __float_as_uint(fa_softcap_full(__uint_as_float(raw[c >> 5][c & 31]), cap));
+                    }
+                }
                 if (edge) {
 #pragma unroll
                     for (int c = 0; c < FB_BN; ++c) {
@@ -1101,14 +1146,14 @@ KB_EXPORT int kb_attention_prefill_tc5_splits(int D, int Hq, int num_tiles, int 
     return splits < 2 ? 1 : (int)splits;
 }
 
-template <int D>
+template <int D, bool CAP>
 static int launch_fa(const CUtensorMap* mq, const CUtensorMap* mk, const CUtensorMap* mv, __nv_bfloat16* out, int out_stride,
                      const int* qo_indptr, const int* seq_lens, const int* block_table, int max_pages, const int* tile_rows,
                      const int* tile_starts, int num_tiles, int Hq, int Hkv, int page_size, int num_pages, float scale, int window,
                      int merged, int splits, float* part_o, float* part_ml, const float* sinks, const __nv_bfloat16* gate, int gate_stride,
-                     int* flag, cudaStream_t stream) {
+                     const KbSoftcap& cap, int* flag, cudaStream_t stream) {
     const size_t smem = FaCfg<D>::SMEM;
-    cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc5_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc5_kernel<D, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     int shift = 0;
     while ((1 << shift) < page_size) ++shift;  // page_size is a power of two here
@@ -1118,9 +1163,9 @@ static int launch_fa(const CUtensorMap* mq, const CUtensorMap* mk, const CUtenso
     const long long single = (long long)Hq * num_tiles;
     const int paired = splits == 1 && num_tiles > 1 && single > resident && (long long)Hq * ((num_tiles + 1) / 2) <= resident ? 1 : 0;
     dim3 grid(Hq, paired ? (num_tiles + 1) / 2 : num_tiles, splits);
-    kb_launch(attention_prefill_tc5_kernel<D>, dim3(grid), dim3(FA_THREADS), smem, stream, *mq, *mk, *mv, out, out_stride, qo_indptr,
+    kb_launch(attention_prefill_tc5_kernel<D, CAP>, dim3(grid), dim3(FA_THREADS), smem, stream, *mq, *mk, *mv, out, out_stride, qo_indptr,
               seq_lens, block_table, max_pages, tile_rows, tile_starts, num_tiles, Hq, Hkv, page_size, shift, num_pages, scale, window, merged,
-              paired, splits, part_o, part_ml, sinks, gate, gate_stride, flag);
+              paired, splits, part_o, part_ml, sinks, gate, gate_stride, cap, flag);
     int rc = kb_launch_result();
     if (rc != 0 || splits == 1) return rc;
     const long long pairs = (long long)num_tiles * FA_BM * Hq;
@@ -1129,18 +1174,20 @@ static int launch_fa(const CUtensorMap* mq, const CUtensorMap* mk, const CUtenso
     return kb_launch_result();
 }
 
+template <bool CAP>
 static int launch_two(const CUtensorMap* mq, const CUtensorMap* mk, const CUtensorMap* mv, __nv_bfloat16* out, int out_stride,
                       const int* qo_indptr, const int* seq_lens, const int* block_table, int max_pages, const int* wide_rows,
                       const int* wide_starts, int num_wide, int Hq, int Hkv, int page_size, int num_pages, float scale, int window,
-                      int merged, const float* sinks, const __nv_bfloat16* gate, int gate_stride, int* flag, cudaStream_t stream) {
-    cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc5_two_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)FbCfg::SMEM);
+                      int merged, const float* sinks, const __nv_bfloat16* gate, int gate_stride, const KbSoftcap& cap, int* flag,
+                      cudaStream_t stream) {
+    cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc5_two_kernel<CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)FbCfg::SMEM);
     if (e != cudaSuccess) return (int)e;
     int shift = 0;
     while ((1 << shift) < page_size) ++shift;
     dim3 grid(Hq, num_wide);
-    kb_launch(attention_prefill_tc5_two_kernel, dim3(grid), dim3(FB_THREADS), FbCfg::SMEM, stream, *mq, *mk, *mv, out, out_stride, qo_indptr,
+    kb_launch(attention_prefill_tc5_two_kernel<CAP>, dim3(grid), dim3(FB_THREADS), FbCfg::SMEM, stream, *mq, *mk, *mv, out, out_stride, qo_indptr,
               seq_lens, block_table, max_pages, wide_rows, wide_starts, num_wide, Hq, Hkv, page_size, shift, num_pages, scale, window, merged,
-              sinks, gate, gate_stride, flag);
+              sinks, gate, gate_stride, cap, flag);
     return kb_launch_result();
 }
 
@@ -1179,13 +1226,14 @@ KB_EXPORT int kb_attention_prefill_tc5_merged(int D, int page_size) { return D >
 // portions go to the kernel that takes two query tiles a block, whose list (wide_rows, wide_starts,
 // num_wide) holds 256 queries per tile.  sinks (optional): one fp32 logit a query head whose exp joins the
 // softmax's denominator; gate (optional): bf16 [tokens, gate_stride], 16-byte aligned rows laid out as out's, by
-// whose sigmoid the result is multiplied.
+// whose sigmoid the result is multiplied.  softcap (optional): a host KbSoftcap (softcap.cuh).
 KB_EXPORT int kb_attention_prefill_tc5(const void* map_q, const void* map_k, const void* map_v, void* out, int out_stride,
                                        const int* qo_indptr, const int* seq_lens, const int* block_table, int max_pages,
                                        const int* tile_rows, const int* tile_starts, int num_tiles, int Hq, int Hkv, int D,
                                        int page_size, int num_pages, float scale, int window, int splits, float* part_o,
                                        float* part_ml, const int* wide_rows, const int* wide_starts, int num_wide, int two_tiles,
-                                       const float* sinks, const void* gate, int gate_stride, int* flag, cudaStream_t stream) {
+                                       const float* sinks, const void* gate, int gate_stride, const void* softcap, int* flag,
+                                       cudaStream_t stream) {
     if (num_tiles == 0) return 0;
     if (gate && (gate_stride % 8 != 0 || ((uintptr_t)gate % 16) != 0)) return KB_ERR_BAD_ARG;  // 16-byte loads beside the stores
     if (two_tiles && (D != 128 || splits != 1 || !wide_rows || !wide_starts || num_wide < 1 || num_wide > 65535)) return KB_ERR_BAD_ARG;
@@ -1196,12 +1244,17 @@ KB_EXPORT int kb_attention_prefill_tc5(const void* map_q, const void* map_k, con
     if (!kb_attention_prefill_tc5_supported(D, page_size)) return KB_ERR_UNSUPPORTED_SIZE;
 #define ARGS (const CUtensorMap*)map_q, (const CUtensorMap*)map_k, (const CUtensorMap*)map_v, (__nv_bfloat16*)out, out_stride, qo_indptr, \
              seq_lens, block_table, max_pages, tile_rows, tile_starts, num_tiles, Hq, Hkv, page_size, num_pages, scale, window,            \
-             kb_attention_prefill_tc5_merged(D, page_size), splits, part_o, part_ml, sinks, (const __nv_bfloat16*)gate, gate_stride, flag, stream
-    if (two_tiles)
-        return launch_two((const CUtensorMap*)map_q, (const CUtensorMap*)map_k, (const CUtensorMap*)map_v, (__nv_bfloat16*)out, out_stride,
-                          qo_indptr, seq_lens, block_table, max_pages, wide_rows, wide_starts, num_wide, Hq, Hkv, page_size, num_pages, scale,
-                          window, kb_attention_prefill_tc5_merged(D, page_size), sinks, (const __nv_bfloat16*)gate, gate_stride, flag, stream);
-    if (D == 64) return launch_fa<64>(ARGS);
-    return launch_fa<128>(ARGS);
+             kb_attention_prefill_tc5_merged(D, page_size), splits, part_o, part_ml, sinks, (const __nv_bfloat16*)gate, gate_stride, cap, flag, stream
+#define TWO_ARGS (const CUtensorMap*)map_q, (const CUtensorMap*)map_k, (const CUtensorMap*)map_v, (__nv_bfloat16*)out, out_stride,          \
+                 qo_indptr, seq_lens, block_table, max_pages, wide_rows, wide_starts, num_wide, Hq, Hkv, page_size, num_pages, scale,      \
+                 window, kb_attention_prefill_tc5_merged(D, page_size), sinks, (const __nv_bfloat16*)gate, gate_stride, cap, flag, stream
+    const KbSoftcap cap = kb_softcap_of(softcap);
+    if (cap.mode != KB_SOFTCAP_NONE) {
+        if (two_tiles) return launch_two<true>(TWO_ARGS);
+        return D == 64 ? launch_fa<64, true>(ARGS) : launch_fa<128, true>(ARGS);
+    }
+    if (two_tiles) return launch_two<false>(TWO_ARGS);
+    return D == 64 ? launch_fa<64, false>(ARGS) : launch_fa<128, false>(ARGS);
+#undef TWO_ARGS
 #undef ARGS
 }

@@ -150,11 +150,11 @@ KB_EXPORT int kb_patch_tokens(int* ids, const int* source, const int* sampled, i
 
 // ------------------------------------------------------------------ RMSNorm
 // One block per output row r; source row s = rows ? rows[r] : r.
-//   v = x[s] (+ delta[s]);  if write_back: x[s] = v  (the fp32 residual sum)
+//   v = x[s] (+ delta[s], or + delta_scale * delta[s] column by column);  if write_back: x[s] = v  (the fp32 residual sum)
 //   out[r] = v * rsqrt(mean(v^2) + eps) * w          (kairyu/models/layers.py:42-46,
 // without its intermediate rounding of the normalised value: one rounding at the end).
 template <typename TX, typename TA, typename TW>
-__global__ void rmsnorm_kernel(TX* __restrict__ x, const TA* __restrict__ delta,
+__global__ void rmsnorm_kernel(TX* __restrict__ x, const TA* __restrict__ delta, const float* __restrict__ delta_scale,
                                const TW* __restrict__ w, TA* __restrict__ out,
                                const int* __restrict__ rows, int H, float eps, int write_back) {
     pdl_wait();
@@ -167,7 +167,7 @@ __global__ void rmsnorm_kernel(TX* __restrict__ x, const TA* __restrict__ delta,
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         float v = to_float(xr[i]);
         if (dr) {
-            v += to_float(dr[i]);
+            v += delta_scale ? to_float(dr[i]) * delta_scale[i] : to_float(dr[i]);
             if (write_back) xr[i] = from_float<TX>(v);
         }
         ss += v * v;
@@ -177,7 +177,7 @@ __global__ void rmsnorm_kernel(TX* __restrict__ x, const TA* __restrict__ delta,
     TA* orow = out + (size_t)r * H;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         float v = to_float(xr[i]);
-        if (dr && !write_back) v += to_float(dr[i]);
+        if (dr && !write_back) v += delta_scale ? to_float(dr[i]) * delta_scale[i] : to_float(dr[i]);
         orow[i] = from_float<TA>(v * inv * to_float(w[i]));
     }
 }
@@ -277,7 +277,7 @@ KB_EXPORT int kb_activation(const void* x, void* y, int is_bf16, long long total
 // chunks in one thread; a larger block (a few rows: every load in flight at once) passes the chunks' sums
 // through shared memory.  Either way a row's result depends on its width alone.
 template <typename TX, typename TA, typename TW>
-__global__ void rmsnorm_vec_kernel(TX* __restrict__ x, const TA* __restrict__ delta,
+__global__ void rmsnorm_vec_kernel(TX* __restrict__ x, const TA* __restrict__ delta, const float* __restrict__ delta_scale,
                                    const TW* __restrict__ w, TA* __restrict__ out,
                                    const int* __restrict__ rows, int H, float eps, int write_back, int groups) {
     pdl_trigger();
@@ -300,6 +300,12 @@ __global__ void rmsnorm_vec_kernel(TX* __restrict__ x, const TA* __restrict__ de
             if (dr) {
                 float d[4];
                 Vec4<TA>::load(dr + 4 * chunk, d);
+                if (delta_scale) {
+                    float by[4];
+                    Vec4<float>::load(delta_scale + 4 * chunk, by);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) d[e] *= by[e];
+                }
 #pragma unroll
                 for (int e = 0; e < 4; ++e) v[c][e] += d[e];
                 if (write_back) Vec4<TX>::store(xr + 4 * chunk, v[c]);
@@ -343,11 +349,11 @@ __global__ void rmsnorm_vec_kernel(TX* __restrict__ x, const TA* __restrict__ de
 }
 
 template <typename TX, typename TA>
-static int rmsnorm_dispatch_w(void* x, const void* delta, const void* w, int w_bf16, void* out,
+static int rmsnorm_dispatch_w(void* x, const void* delta, const float* delta_scale, const void* w, int w_bf16, void* out,
                               const int* rows, int R, int H, float eps, int write_back,
                               cudaStream_t stream) {
     const bool aligned = ((uintptr_t)x % 16 == 0) && ((uintptr_t)out % 16 == 0) && ((uintptr_t)w % 16 == 0) &&
-                         (delta == nullptr || (uintptr_t)delta % 16 == 0);
+                         (delta == nullptr || (uintptr_t)delta % 16 == 0) && (uintptr_t)delta_scale % 16 == 0;
     if (H % 4 == 0 && H <= 16 * 1024 && aligned) {
         // Many rows (a prompt portion): blocks that hold every chunk a thread may, so that an SM has eight
         // small blocks in different phases (loads, the sum, stores) instead of two large ones in step (2,048
@@ -364,24 +370,25 @@ static int rmsnorm_dispatch_w(void* x, const void* delta, const void* w, int w_b
         }
         if (w_bf16)
             kb_launch(rmsnorm_vec_kernel<TX, TA, __nv_bfloat16>, dim3(R), dim3(threads_v), 0, stream, 
-                (TX*)x, (const TA*)delta, (const __nv_bfloat16*)w, (TA*)out, rows, H, eps, write_back, groups);
+                (TX*)x, (const TA*)delta, delta_scale, (const __nv_bfloat16*)w, (TA*)out, rows, H, eps, write_back, groups);
         else
             kb_launch(rmsnorm_vec_kernel<TX, TA, float>, dim3(R), dim3(threads_v), 0, stream, 
-                (TX*)x, (const TA*)delta, (const float*)w, (TA*)out, rows, H, eps, write_back, groups);
+                (TX*)x, (const TA*)delta, delta_scale, (const float*)w, (TA*)out, rows, H, eps, write_back, groups);
         return kb_launch_result();
     }
     const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
     if (w_bf16)
         kb_launch(rmsnorm_kernel<TX, TA, __nv_bfloat16>, dim3(R), dim3(threads), 0, stream, 
-            (TX*)x, (const TA*)delta, (const __nv_bfloat16*)w, (TA*)out, rows, H, eps, write_back);
+            (TX*)x, (const TA*)delta, delta_scale, (const __nv_bfloat16*)w, (TA*)out, rows, H, eps, write_back);
     else
         kb_launch(rmsnorm_kernel<TX, TA, float>, dim3(R), dim3(threads), 0, stream, 
-            (TX*)x, (const TA*)delta, (const float*)w, (TA*)out, rows, H, eps, write_back);
+            (TX*)x, (const TA*)delta, delta_scale, (const float*)w, (TA*)out, rows, H, eps, write_back);
     return kb_launch_result();
 }
 
-// x: [*, H] fp32 or bf16 (x_bf16); delta/out: activation dtype (act_bf16); w: fp32 or bf16.
-KB_EXPORT int kb_rmsnorm(void* x, int x_bf16, const void* delta, const void* w, int w_bf16,
+// x: [*, H] fp32 or bf16 (x_bf16); delta/out: activation dtype (act_bf16); delta_scale: null, or a factor a column of delta;
+// w: fp32 or bf16.
+KB_EXPORT int kb_rmsnorm(void* x, int x_bf16, const void* delta, const float* delta_scale, const void* w, int w_bf16,
                          void* out, int act_bf16, const int* rows, int R, int H, float eps,
                          int write_back, cudaStream_t stream) {
     if (R == 0) return 0;
@@ -390,12 +397,12 @@ KB_EXPORT int kb_rmsnorm(void* x, int x_bf16, const void* delta, const void* w, 
     if (rows) write_back = 0;
     if (x_bf16) {
         if (act_bf16)
-            return rmsnorm_dispatch_w<__nv_bfloat16, __nv_bfloat16>(x, delta, w, w_bf16, out, rows, R, H, eps, write_back, stream);
+            return rmsnorm_dispatch_w<__nv_bfloat16, __nv_bfloat16>(x, delta, delta_scale, w, w_bf16, out, rows, R, H, eps, write_back, stream);
         return KB_ERR_BAD_ARG;  // bf16 input with fp32 activations is not a mode of this engine
     }
     if (act_bf16)
-        return rmsnorm_dispatch_w<float, __nv_bfloat16>(x, delta, w, w_bf16, out, rows, R, H, eps, write_back, stream);
-    return rmsnorm_dispatch_w<float, float>(x, delta, w, w_bf16, out, rows, R, H, eps, write_back, stream);
+        return rmsnorm_dispatch_w<float, __nv_bfloat16>(x, delta, delta_scale, w, w_bf16, out, rows, R, H, eps, write_back, stream);
+    return rmsnorm_dispatch_w<float, float>(x, delta, delta_scale, w, w_bf16, out, rows, R, H, eps, write_back, stream);
 }
 
 // ------------------------------------------------------------------ SiLU(gate) * up
@@ -507,5 +514,50 @@ KB_EXPORT int kb_scaled_sum(const void* a, float sa, const void* b, float sb, vo
         kb_launch(scaled_sum_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)a, sa, (const __nv_bfloat16*)b, sb, (__nv_bfloat16*)out, (size_t)n);
     else
         kb_launch(scaled_sum_kernel<float>, grid, dim3(256), 0, stream, (const float*)a, sa, (const float*)b, sb, (float*)out, (size_t)n);
+    return kb_launch_result();
+}
+
+// ------------------------------------------------------------------ output gate
+// x[t, c] *= sigmoid(gate[t, c]) in place, 32-bit with one rounding; the gate's rows may be part of wider ones.
+template <typename T>
+__global__ void __launch_bounds__(256) sigmoid_gate_kernel(T* __restrict__ x, const T* __restrict__ gate, int gate_stride, int C) {
+    pdl_trigger();
+    pdl_wait();
+    T* row = x + (size_t)blockIdx.y * C;
+    const T* g = gate + (size_t)blockIdx.y * gate_stride;
+    for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < C; c += gridDim.x * blockDim.x)
+        row[c] = from_float<T>(to_float(row[c]) / (1.0f + expf(-to_float(g[c]))));
+}
+
+// four columns a thread a turn, for rows of whole groups of four on aligned places
+template <typename T>
+__global__ void __launch_bounds__(256) sigmoid_gate_vec_kernel(T* __restrict__ x, const T* __restrict__ gate, int gate_stride, int C) {
+    pdl_trigger();
+    pdl_wait();
+    T* row = x + (size_t)blockIdx.y * C;
+    const T* g = gate + (size_t)blockIdx.y * gate_stride;
+    for (int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4; c < C; c += gridDim.x * blockDim.x * 4) {
+        float v[4], by[4];
+        Vec4<T>::load(row + c, v);
+        Vec4<T>::load(g + c, by);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[e] /= 1.0f + expf(-by[e]);
+        Vec4<T>::store(row + c, v);
+    }
+}
+
+KB_EXPORT int kb_sigmoid_gate(void* x, const void* gate, int gate_stride, int is_bf16, int rows, int C, cudaStream_t stream) {
+    if (rows == 0 || C == 0) return 0;
+    if (!x || !gate) return KB_ERR_NULL;
+    if (rows > 65535) return KB_ERR_UNSUPPORTED_SIZE;
+    const bool vec = C % 4 == 0 && gate_stride % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)gate % (is_bf16 ? 8 : 16) == 0;
+    const dim3 grid(((vec ? C / 4 : C) + 255) / 256, rows);
+#define LAUNCH(KERNEL, TT) kb_launch(KERNEL<TT>, grid, dim3(256), 0, stream, (TT*)x, (const TT*)gate, gate_stride, C)
+    if (is_bf16) {
+        if (vec) LAUNCH(sigmoid_gate_vec_kernel, __nv_bfloat16); else LAUNCH(sigmoid_gate_kernel, __nv_bfloat16);
+    } else {
+        if (vec) LAUNCH(sigmoid_gate_vec_kernel, float); else LAUNCH(sigmoid_gate_kernel, float);
+    }
+#undef LAUNCH
     return kb_launch_result();
 }

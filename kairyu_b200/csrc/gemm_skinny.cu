@@ -16,7 +16,8 @@
 // norm, kairyu/models/llama.py:88-101 the residual arrangement).  With y = rmsnorm(r) * g feeding
 // a product, (y . W^T)[m] = rstd[m] * ((r[m] * g) . W^T): the product before can leave r * g
 // (rounded to bf16) and the sum of r^2, and this product scales its rows by rstd in the epilogue.
-//   * fold:  the epilogue adds the result to the fp32 residual r (in place), writes bf16(r * g)
+//   * fold:  the epilogue adds the result (times a factor a column, for a model that scales what it adds) to the
+//     fp32 residual r (in place), writes bf16(r * g)
 //     for the next product and, per block, the partial sums of r^2 over the block's columns;
 //   * scale: the epilogue multiplies row m by rsqrt(sum of the partial sums / H + eps) before
 //     bias and gate.  The partial sums are added in block order, so the result does not depend
@@ -48,9 +49,10 @@ struct SkinnyFusion {
     int in_blocks;
     float in_inv_hidden;
     float in_eps;
-    // fold: residual[m, n] += result; values[m, n] = bf16(residual * norm_w[n]); out_sumsq[block * 16 + m]
+    // fold: residual[m, n] += result (* fold_scale[n] where that is given); values[m, n] = bf16(residual * norm_w[n]); out_sumsq[block * 16 + m]
     float* residual;
     int ldr;
+    const float* fold_scale;
     const void* norm_w;
     int norm_w_bf16;
     __nv_bfloat16* values;
@@ -263,13 +265,14 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bflo
         for (int i = 0; i < SUM_ROUNDS; ++i) my_sum += part[i];
     }
     // fold: this thread's element of the residual and of the norm weight, asked for now and used in the epilogue
-    float held_residual = 0.0f, held_weight = 0.0f;
+    float held_residual = 0.0f, held_weight = 0.0f, held_scale = 1.0f;
     if (FUSED && fusion.residual != nullptr && threadIdx.x < NT * 8 * 16) {
         const int r = threadIdx.x & 15;
         const int token = threadIdx.x >> 4;
         const int n = column_of(r);
         if (token < M && r < rows_per_block && n < rows_out) {
             held_residual = fusion.residual[(size_t)token * fusion.ldr + n];
+            if (fusion.fold_scale) held_scale = fusion.fold_scale[n];
             held_weight = fusion.norm_w_bf16 ? __bfloat162float(((const __nv_bfloat16*)fusion.norm_w)[n]) : ((const float*)fusion.norm_w)[n];
         }
     }
@@ -357,7 +360,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bflo
         float square = 0.0f;
         if (valid) {
             // (NT * 8 * 16 <= SK_THREADS: the loop runs once and idx == threadIdx.x, as when the values were fetched)
-            const float sum = held_residual + result;
+            const float sum = held_residual + result * held_scale;
             fusion.residual[(size_t)token * fusion.ldr + n] = sum;
             fusion.values[(size_t)token * fusion.ldv + n] = __float2bfloat16_rn(sum * held_weight);
             square = sum * sum;
@@ -479,10 +482,10 @@ KB_EXPORT int kb_gemm_skinny_max_sum_blocks() { return SK_SUM_BLOCKS; }
 // in_sumsq (or null): the producer's partial sums [in_blocks, 16]; rows are scaled by
 //   rsqrt(sum / in_hidden + in_eps) before bias and gate.
 // residual (or null; not with gated): [M, N] fp32, row stride ldr; the result is added to it in
-//   place, values[M, N] = bf16(residual * norm_w) and out_sumsq[blocks, 16] are written; out is not.
+//   place (times fold_scale[N], fp32, where that is given), values[M, N] = bf16(residual * norm_w) and out_sumsq[blocks, 16] are written; out is not.
 KB_EXPORT int kb_gemm_skinny_fused(const void* x, int ldx, const void* w, int ldw, const void* bias, void* out, int out_fp32,
                                    int ldo, int M, int N, int K, int gated, const float* in_sumsq, int in_blocks, int in_hidden,
-                                   float in_eps, float* residual, int ldr, const void* norm_w, int norm_w_bf16, void* values,
+                                   float in_eps, float* residual, int ldr, const float* fold_scale, const void* norm_w, int norm_w_bf16, void* values,
                                    int ldv, float* out_sumsq, cudaStream_t stream) {
     SkinnyFusion fusion = {};
     fusion.in_sumsq = in_sumsq;
@@ -491,6 +494,7 @@ KB_EXPORT int kb_gemm_skinny_fused(const void* x, int ldx, const void* w, int ld
     fusion.in_eps = in_eps;
     fusion.residual = residual;
     fusion.ldr = ldr;
+    fusion.fold_scale = fold_scale;
     fusion.norm_w = norm_w;
     fusion.norm_w_bf16 = norm_w_bf16;
     fusion.values = (__nv_bfloat16*)values;

@@ -8,6 +8,10 @@
 //   q goes back in place, k to the key page [pages, page_size, Hkv, D], v (untouched) to the value
 //   page [pages, page_size, Hkv, DV]
 //
+// With statistics a head (per_head: weights of D entries that the heads share) the norm may also come BEHIND the
+// rotation (norm_after): every turned head of q and k is divided by its own root mean square, without a weight.
+// v_offset may be k_offset: a value is then the key as projected.
+//
 // Statistics, weights and the rotation are 32-bit, with one rounding at the store.  One block per
 // token; a thread owns whole pairs, so the in-place write of q races with nothing.  Positions below
 // write_from[row] lie in pages the request only reads and are skipped (q is still produced).
@@ -20,7 +24,7 @@
 template <typename T, typename TW>
 __global__ void __launch_bounds__(PR_THREADS)
 projection_norm_rope_write_kernel(T* __restrict__ packed, int stride, int k_offset, int v_offset, int Hq, int Hkv, int D, int DV,
-                                  const TW* __restrict__ wq, const TW* __restrict__ wk, float eps, int per_head,
+                                  const TW* __restrict__ wq, const TW* __restrict__ wk, float eps, int per_head, int norm_after,
                                   const float* __restrict__ cos_table, const float* __restrict__ sin_table, int rot_half, int max_pos,
                                   int interleaved, const float* __restrict__ v_cos, const float* __restrict__ v_sin, int v_rot_half, const int* __restrict__ positions, const int* __restrict__ row_ids,
                                   const int* __restrict__ block_table, int max_pages, const int* __restrict__ write_from,
@@ -65,7 +69,7 @@ projection_norm_rope_write_kernel(T* __restrict__ packed, int stride, int k_offs
     // a head is rot_half pairs and D - 2 * rot_half single columns: D - rot_half units
     const int units = D - rot_half;
     // one unit of head `head`: normed by inv and the weight at w_first + column, rotated, stored
-    auto unit = [&](int head, int i, float inv, int w_first) {
+    auto unit = [&](int head, int i, float inv, int w_first, float behind) {
         const bool is_q = head < Hq;
         const int first = (is_q ? head : head - Hq) * D;
         const T* src = (is_q ? q : k) + first;
@@ -79,12 +83,12 @@ projection_norm_rope_write_kernel(T* __restrict__ packed, int stride, int k_offs
             float rx, ry;
             rotate(x, y, cs[i], sn[i], rx, ry);
             if (dst) {
-                dst[a] = from_float<T>(pos_ok ? rx : 0.0f);
-                dst[b] = from_float<T>(pos_ok ? ry : 0.0f);
+                dst[a] = from_float<T>(pos_ok ? rx * behind : 0.0f);
+                dst[b] = from_float<T>(pos_ok ? ry * behind : 0.0f);
             }
         } else if (dst) {
             const int c = i + rot_half;
-            dst[c] = from_float<T>(to_float(src[c]) * inv * (w ? to_float(w[w_first + c]) : 1.0f));
+            dst[c] = from_float<T>(to_float(src[c]) * inv * (w ? to_float(w[w_first + c]) : 1.0f) * behind);
         }
     };
     if (per_head) {
@@ -101,7 +105,25 @@ projection_norm_rope_write_kernel(T* __restrict__ packed, int stride, int k_offs
                 }
                 inv = rsqrtf(warp_sum(ss) / (float)D + eps);  // the butterfly also orders these reads before the writes below
             }
-            for (int i = lane; i < units; i += 32) unit(head, i, inv, 0);
+            float behind = 1.0f;
+            if (norm_after) {
+                const T* src = head < Hq ? q + head * D : k + (head - Hq) * D;
+                float ss = 0.0f;
+                for (int i = lane; i < units; i += 32) {
+                    if (i < rot_half) {
+                        int a, b;
+                        rotary_pair(i, rot_half, interleaved, a, b);
+                        float rx, ry;
+                        rotate(to_float(src[a]), to_float(src[b]), cs[i], sn[i], rx, ry);
+                        ss += rx * rx + ry * ry;
+                    } else {
+                        const float x = to_float(src[i + rot_half]);
+                        ss += x * x;
+                    }
+                }
+                behind = rsqrtf(warp_sum(ss) / (float)D + eps);
+            }
+            for (int i = lane; i < units; i += 32) unit(head, i, inv, 0, behind);
         }
     } else {
         float inv_q = 1.0f, inv_k = 1.0f;
@@ -120,7 +142,7 @@ projection_norm_rope_write_kernel(T* __restrict__ packed, int stride, int k_offs
         }
         for (int u = threadIdx.x; u < (Hq + Hkv) * units; u += blockDim.x) {
             const int head = u / units;
-            unit(head, u % units, head < Hq ? inv_q : inv_k, (head < Hq ? head : head - Hq) * D);
+            unit(head, u % units, head < Hq ? inv_q : inv_k, (head < Hq ? head : head - Hq) * D, 1.0f);
         }
     }
     if (v_dst && v_rot_half > 0) {
@@ -373,11 +395,145 @@ projection_norm_rope_write_vec_kernel(__nv_bfloat16* __restrict__ packed, int st
     }
 }
 
+// The same with statistics a head, or none, on bfloat16 rows of whole 16-byte groups: GROUP lanes hold a head in registers
+// (eight columns a lane), so a head is read once, its sum is a butterfly among its lanes and nothing waits for another head.
+// A value head is an item of its own, or (values that are the keys as projected) goes out with its key.
+template <int GROUP, typename TW>
+__global__ void __launch_bounds__(PR_THREADS)
+head_norm_rope_write_kernel(__nv_bfloat16* __restrict__ packed, int stride, int k_offset, int v_offset, int Hq, int Hkv, int D, int DV,
+                            const TW* __restrict__ wq, const TW* __restrict__ wk, float eps, int norm_after,
+                            const float* __restrict__ cos_table, const float* __restrict__ sin_table, int rot_half, int max_pos,
+                            int interleaved, const int* __restrict__ positions, const int* __restrict__ row_ids,
+                            const int* __restrict__ block_table, int max_pages, const int* __restrict__ write_from,
+                            __nv_bfloat16* __restrict__ k_cache, __nv_bfloat16* __restrict__ v_cache, int page_size, int num_pages,
+                            int num_rows, int T, int* flag) {
+    pdl_trigger();
+    const bool keys_are_values = v_offset == k_offset && DV == D;
+    const int heads = Hq + Hkv + (k_cache && !keys_are_values ? Hkv : 0);
+    const long long item = ((long long)blockIdx.x * PR_THREADS + threadIdx.x) / GROUP;
+    const int j = threadIdx.x % GROUP;  // this lane's eight columns of the head
+    const bool live = item < (long long)T * heads;
+    const int t = live ? (int)(item / heads) : 0;
+    const int head = live ? (int)(item % heads) : 0;
+    const bool is_q = head < Hq, is_v = head >= Hq + Hkv;
+    const int pos = positions[t];
+    const bool pos_ok = rot_half == 0 || (pos >= 0 && pos < max_pos);
+    // where a key or value row goes (negative: nowhere)
+    long long place = -1;
+    int trouble = pos_ok ? 0 : KB_FLAG_BAD_POS;
+    if (!is_q && k_cache) {
+        const int row = row_ids[t];
+        if (row < 0 || row >= num_rows) {
+            trouble |= KB_FLAG_BAD_ROW;
+        } else if (!(write_from && pos < write_from[row])) {
+            const int page_index = pos / page_size;
+            const int page = (pos >= 0 && page_index < max_pages) ? block_table[(size_t)row * max_pages + page_index] : -1;
+            if (page < 0 || page >= num_pages) trouble |= KB_FLAG_BAD_PAGE;
+            else place = (long long)page * page_size + (pos % page_size);
+        }
+    }
+    const int groups = (is_v ? DV : D) / 8;
+    const bool holds = live && j < groups;
+    // this lane's angles: of pair (i, i + rot_half) for both of the lanes that hold its two sides; of four pairs when interleaved
+    const int rot_groups = interleaved ? rot_half / 4 : rot_half / 8;
+    const bool turns = holds && !is_v && j < (interleaved ? rot_groups : 2 * rot_groups);
+    float c8[8], s8[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+        c8[e] = 1.0f;
+        s8[e] = 0.0f;
+    }
+    if (turns && pos_ok) {
+        const float* cs = cos_table + (size_t)pos * rot_half;
+        const float* sn = sin_table + (size_t)pos * rot_half;
+        if (interleaved) {
+            load_floats(cs + j * 4, 4, c8);
+            load_floats(sn + j * 4, 4, s8);
+        } else {
+            load_floats(cs + (j % rot_groups) * 8, 8, c8);
+            load_floats(sn + (j % rot_groups) * 8, 8, s8);
+        }
+    }
+    pdl_wait();
+    if (live && j == 0 && trouble && flag) atomicOr(flag, trouble);
+    const int local = is_q ? head : (is_v ? head - Hq - Hkv : head - Hq);
+    __nv_bfloat16* src = packed + (size_t)t * stride + (is_q ? 0 : is_v ? v_offset : k_offset) + local * (is_v ? DV : D) + j * 8;
+    Bf16x8 raw;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) raw.v[e] = __floats2bfloat162_rn(0.0f, 0.0f);
+    if (holds) raw = *reinterpret_cast<const Bf16x8*>(src);
+    float a[8];
+    unpack8(raw, a);
+    auto sum_of_squares = [&]() -> float {
+        float ss = 0.0f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss += a[e] * a[e];
+#pragma unroll
+        for (int offset = GROUP / 2; offset > 0; offset >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, offset);
+        return ss;
+    };
+    if (wq) {
+        const float inv = rsqrtf(sum_of_squares() / (float)D + eps);
+        if (holds && !is_v) {
+            float w8[8];
+            load_weights8(is_q ? wq : wk, j * 8, inv, w8);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) a[e] *= w8[e];
+        }
+    }
+    if (interleaved) {
+        if (turns) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                float rx, ry;
+                rotate(a[2 * e], a[2 * e + 1], c8[e], s8[e], rx, ry);
+                a[2 * e] = rx;
+                a[2 * e + 1] = ry;
+            }
+        }
+    } else if (rot_half > 0) {
+        // the lane that holds the other side of these pairs; lanes that turn nothing exchange with themselves
+        const bool first = j < rot_groups;
+        const int lane = threadIdx.x & 31;
+        const int partner = turns ? lane + (first ? rot_groups : -rot_groups) : lane;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            const float other = __shfl_sync(0xffffffffu, a[e], partner);
+            float rx, ry;
+            rotate(first ? a[e] : other, first ? other : a[e], c8[e], s8[e], rx, ry);
+            if (turns) a[e] = first ? rx : ry;
+        }
+    }
+    if (norm_after) {
+        const float inv = rsqrtf(sum_of_squares() / (float)D + eps);
+        if (!is_v) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) a[e] *= inv;
+        }
+    }
+    if (!holds) return;
+    if (turns && !pos_ok) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) a[e] = 0.0f;
+    }
+    if (is_q) {
+        *reinterpret_cast<Bf16x8*>(src) = pack8(a);
+    } else if (place >= 0) {
+        if (is_v) {
+            *reinterpret_cast<Bf16x8*>(v_cache + ((size_t)place * Hkv + local) * DV + j * 8) = raw;
+        } else {
+            *reinterpret_cast<Bf16x8*>(k_cache + ((size_t)place * Hkv + local) * D + j * 8) = pack8(a);
+            if (keys_are_values) *reinterpret_cast<Bf16x8*>(v_cache + ((size_t)place * Hkv + local) * D + j * 8) = raw;
+        }
+    }
+}
+
 // wq/wk null: no norm; per_head: statistics a head and weights of D entries, else over the whole projection.
+// norm_after (with per_head and without weights): every turned head of q and k divided by its root mean square.
 // cos/sin null (rot_half 0): no rotation.  v_cos/v_sin (v_rot_half > 0): the values turn too, by a table of their
 // own of the same number of positions.  k_cache null: q only.
 KB_EXPORT int kb_projection_norm_rope_write(void* packed, int stride, int is_bf16, int T, int k_offset, int v_offset, int Hq, int Hkv,
-                                            int D, int DV, const void* wq, const void* wk, int w_bf16, float eps, int per_head,
+                                            int D, int DV, const void* wq, const void* wk, int w_bf16, float eps, int per_head, int norm_after,
                                             const float* cos_table, const float* sin_table, int rot_half, int max_pos, int interleaved,
                                             const float* v_cos, const float* v_sin, int v_rot_half,
                                             const int* positions, const int* row_ids, const int* block_table, int max_pages,
@@ -386,13 +542,14 @@ KB_EXPORT int kb_projection_norm_rope_write(void* packed, int stride, int is_bf1
     if (T == 0) return 0;
     if (!packed || !positions || !row_ids) return KB_ERR_NULL;
     if ((wq == nullptr) != (wk == nullptr)) return KB_ERR_BAD_ARG;
+    if (norm_after && (!per_head || wq)) return KB_ERR_BAD_ARG;
     if (Hq < 1 || Hkv < 0 || (Hkv == 0 && k_cache) || D < 1 || DV < 1 || rot_half < 0 || 2 * rot_half > D) return KB_ERR_BAD_ARG;  // no key heads: queries alone
     if (rot_half > 0 && (!cos_table || !sin_table || max_pos < 1)) return KB_ERR_NULL;
     if (v_rot_half < 0 || 2 * v_rot_half > DV || (v_rot_half > 0 && (!v_cos || !v_sin || max_pos < 1))) return KB_ERR_BAD_ARG;
     if (k_cache && (!v_cache || !block_table || page_size < 1)) return KB_ERR_NULL;
 #define LAUNCH(TT, TW)                                                                                                              \
     kb_launch(projection_norm_rope_write_kernel<TT, TW>, dim3(T), dim3(PR_THREADS), 0, stream, (TT*)packed, stride, k_offset,         \
-              v_offset, Hq, Hkv, D, DV, (const TW*)wq, (const TW*)wk, eps, per_head, cos_table, sin_table, rot_half, max_pos,       \
+              v_offset, Hq, Hkv, D, DV, (const TW*)wq, (const TW*)wk, eps, per_head, norm_after, cos_table, sin_table, rot_half, max_pos, \
               interleaved, v_cos, v_sin, v_rot_half, positions, row_ids, block_table, max_pages, write_from, (TT*)k_cache, (TT*)v_cache, page_size, num_pages, num_rows, flag)
     // whole 16-byte groups everywhere: heads, offsets, rows, the rotated part (split halves: each half) and the pages
     const bool groups_of_eight = (!per_head || Hq + Hkv <= PR_MAX_HEADS) && (v_rot_half == 0 || (interleaved && v_rot_half % 4 == 0 && (uintptr_t)v_cos % 16 == 0 && (uintptr_t)v_sin % 16 == 0)) && is_bf16 && D % 8 == 0 && DV % 8 == 0 && stride % 8 == 0 && k_offset % 8 == 0 && v_offset % 8 == 0 &&
@@ -404,7 +561,21 @@ KB_EXPORT int kb_projection_norm_rope_write(void* packed, int stride, int is_bf1
               k_offset, v_offset, Hq, Hkv, D, DV, (const TW*)wq, (const TW*)wk, eps, per_head, cos_table, sin_table, rot_half, max_pos, \
               interleaved, v_cos, v_sin, v_rot_half, positions, row_ids, block_table, max_pages, write_from, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, \
               page_size, num_pages, num_rows, flag)
-    if (groups_of_eight) {
+#define LAUNCH_HEADS(GROUP, TW)                                                                                                     \
+    kb_launch(head_norm_rope_write_kernel<GROUP, TW>, dim3((unsigned)((items * GROUP + PR_THREADS - 1) / PR_THREADS)), dim3(PR_THREADS), 0,  \
+              stream, (__nv_bfloat16*)packed, stride, k_offset, v_offset, Hq, Hkv, D, DV, (const TW*)wq, (const TW*)wk, eps, norm_after,  \
+              cos_table, sin_table, rot_half, max_pos, interleaved, positions, row_ids, block_table, max_pages, write_from,         \
+              (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, page_size, num_pages, num_rows, T, flag)
+#define PICK_HEADS(TW)                                                                                                              \
+    do {                                                                                                                            \
+        if (lanes <= 4) LAUNCH_HEADS(4, TW); else if (lanes <= 8) LAUNCH_HEADS(8, TW);                                              \
+        else if (lanes <= 16) LAUNCH_HEADS(16, TW); else LAUNCH_HEADS(32, TW);                                                      \
+    } while (0)
+    const int lanes = (k_cache && DV > D ? DV : D) / 8;  // 16-byte groups of the widest head
+    const long long items = (long long)T * (Hq + Hkv + (k_cache && !(v_offset == k_offset && DV == D) ? Hkv : 0));
+    if (groups_of_eight && (per_head || !wq) && v_rot_half == 0 && lanes <= 32 && items < (1ll << 27)) {
+        if (w_bf16) PICK_HEADS(__nv_bfloat16); else PICK_HEADS(float);
+    } else if (groups_of_eight && !norm_after) {
         if (w_bf16) LAUNCH_VEC(__nv_bfloat16); else LAUNCH_VEC(float);
     } else if (is_bf16) {
         if (w_bf16) LAUNCH(__nv_bfloat16, __nv_bfloat16); else LAUNCH(__nv_bfloat16, float);
@@ -413,6 +584,8 @@ KB_EXPORT int kb_projection_norm_rope_write(void* packed, int stride, int is_bf1
     }
 #undef LAUNCH
 #undef LAUNCH_VEC
+#undef LAUNCH_HEADS
+#undef PICK_HEADS
     return kb_launch_result();
 }
 

@@ -9,6 +9,7 @@ an error.  Model parts call these as ``kernels.<name>(...)``.
 from __future__ import annotations
 
 import ctypes
+import math
 from dataclasses import dataclass
 from typing import Optional
 
@@ -182,14 +183,15 @@ def rmsnorm(
     out: torch.Tensor,
     *,
     delta: Optional[torch.Tensor] = None,
+    delta_scale: Optional[torch.Tensor] = None,
     rows: Optional[torch.Tensor] = None,
 ) -> None:
-    """``x += delta`` (if given and ``rows`` is None), ``out = rmsnorm(x) * weight``.
+    """``x += delta`` (if given and ``rows`` is None; ``delta_scale``, fp32 [hidden]: ``x += delta_scale * delta``), ``out = rmsnorm(x) * weight``.
 
     With ``rows`` only the listed rows of x (+delta) are normed, into
     out[0..len(rows)), and x is not modified.
     """
-    _need_cuda("rmsnorm", x, weight, out, delta, rows)
+    _need_cuda("rmsnorm", x, weight, out, delta, delta_scale, rows)
     _need_i32("rmsnorm", rows)
     H = x.shape[-1]
     R = rows.numel() if rows is not None else x.shape[0]
@@ -199,9 +201,11 @@ def rmsnorm(
         raise KernelError("rmsnorm: shape mismatch")
     if delta is not None and (delta.dtype != out.dtype or delta.shape != x.shape):
         raise KernelError("rmsnorm: delta must have the activation dtype and x's shape")
-    fn = _fn("elementwise", "kb_rmsnorm", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_int, c_void_p])
+    if delta_scale is not None and (delta is None or delta_scale.dtype != torch.float32 or delta_scale.numel() != H or not delta_scale.is_contiguous()):
+        raise KernelError("rmsnorm: delta's scale must be contiguous fp32, one factor a column")
+    fn = _fn("elementwise", "kb_rmsnorm", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_int, c_void_p])
     _check(
-        fn(x.data_ptr(), _is_bf16(x, "rmsnorm"), _ptr(delta), weight.data_ptr(), _is_bf16(weight, "rmsnorm"), out.data_ptr(), _is_bf16(out, "rmsnorm"), _ptr(rows), R, H, float(eps), 1, _stream()),
+        fn(x.data_ptr(), _is_bf16(x, "rmsnorm"), _ptr(delta), _ptr(delta_scale), weight.data_ptr(), _is_bf16(weight, "rmsnorm"), out.data_ptr(), _is_bf16(out, "rmsnorm"), _ptr(rows), R, H, float(eps), 1, _stream()),
         "rmsnorm",
     )
 
@@ -354,15 +358,18 @@ def projection_norm_rope_write(
     v_cache: Optional[torch.Tensor] = None,
     flag: Optional[torch.Tensor] = None,
     per_head_norm: bool = False,
+    unit_heads: bool = False,
     v_cos: Optional[torch.Tensor] = None,
     v_sin: Optional[torch.Tensor] = None,
 ) -> None:
     """On the packed rows ``[q | ... k at k_offset ... v at v_offset ...]``: RMS norm of q over all its ``heads * dim``
     columns at once and of k over all of its (if weights of those sizes are given; with ``per_head_norm`` the statistics
-    are a head's and the weights ``dim`` entries that the heads share), rotation of the first
+    are a head's and the weights ``dim`` entries that the heads share; with ``unit_heads``, and without weights, every head of
+    q and k is divided by its root mean square behind its rotation), rotation of the first
     ``2 * cos.shape[1]`` columns of every head (pairs (i, i + half), or (2i, 2i + 1) when ``interleaved``), q back in place, k
     into ``k_cache`` [pages, page, kv_heads, dim] and v into ``v_cache`` [pages, page, kv_heads, value_dim]; with ``v_cos`` /
-    ``v_sin`` (tables of as many positions) the first ``2 * v_cos.shape[1]`` columns of every value head turn too."""
+    ``v_sin`` (tables of as many positions) the first ``2 * v_cos.shape[1]`` columns of every value head turn too.
+    ``v_offset`` may be ``k_offset``: a value is then the key as projected."""
     what = "projection_norm_rope_write"
     _need_cuda(what, packed, positions, row_ids, q_norm_weight, k_norm_weight, cos, sin, block_table, write_from, k_cache, v_cache, flag, v_cos, v_sin)
     _need_i32(what, positions, row_ids, block_table, write_from)
@@ -376,6 +383,8 @@ def projection_norm_rope_write(
         max_pos, rot_half = cos.shape
         if 2 * rot_half > head_dim:
             raise KernelError(f"{what}: {2 * rot_half} rotated columns in a head of {head_dim}")
+    if unit_heads and q_norm_weight is not None:
+        raise KernelError(f"{what}: heads of unit mean square behind the rotation come without norm weights")
     v_rot_half = 0
     if v_cos is not None:
         if v_sin is None or v_cos.shape != v_sin.shape or v_cos.dtype != torch.float32 or v_sin.dtype != torch.float32 or not (v_cos.is_contiguous() and v_sin.is_contiguous()):
@@ -405,10 +414,10 @@ def projection_norm_rope_write(
             raise KernelError(f"{what}: a cache write needs the block table")
         num_rows, max_pages = block_table.shape
     fn = _fn("projection_rope", "kb_projection_norm_rope_write",
-             [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p, c_int,
+             [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_int,
               c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p])
     _check(fn(packed.data_ptr(), packed.stride(0), _is_bf16(packed, what), packed.shape[0], int(k_offset), int(v_offset), num_q_heads, num_kv_heads,
-              head_dim, value_dim, _ptr(q_norm_weight), _ptr(k_norm_weight), w_bf16, float(eps), 1 if per_head_norm else 0, _ptr(cos), _ptr(sin),
+              head_dim, value_dim, _ptr(q_norm_weight), _ptr(k_norm_weight), w_bf16, float(eps), 1 if per_head_norm or unit_heads else 0, 1 if unit_heads else 0, _ptr(cos), _ptr(sin),
               rot_half, max_pos, 1 if interleaved else 0, _ptr(v_cos), _ptr(v_sin), v_rot_half, positions.data_ptr(), row_ids.data_ptr(), _ptr(block_table), max_pages, _ptr(write_from), _ptr(k_cache),
               _ptr(v_cache), page_size, num_pages, num_rows, _ptr(flag), _stream()), what)
 
@@ -431,6 +440,16 @@ def rotate_heads(x: torch.Tensor, *, heads: int, head_dim: int, cos: torch.Tenso
              [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p])
     _check(fn(x.data_ptr(), x.stride(0), _is_bf16(x, what), x.shape[0], heads, head_dim, cos.data_ptr(), sin.data_ptr(), rot_half, max_pos,
               1 if interleaved else 0, 1 if inverse else 0, positions.data_ptr(), _ptr(flag), _stream()), what)
+
+
+def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor) -> None:
+    """``x *= sigmoid(gate)``, in place, 32-bit with one rounding.  ``x`` [rows, columns] contiguous; ``gate`` of its shape and dtype,
+    any row stride (a view into wider rows)."""
+    _need_cuda("sigmoid_gate", x, gate)
+    if not x.is_contiguous() or gate.shape != x.shape or gate.dtype != x.dtype or gate.stride(1) != 1:
+        raise KernelError("sigmoid_gate: contiguous rows and a gate of their shape and dtype with unit inner stride")
+    fn = _fn("elementwise", "kb_sigmoid_gate", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(x.data_ptr(), gate.data_ptr(), gate.stride(0), _is_bf16(x, "sigmoid_gate"), x.shape[0], x.shape[1], _stream()), "sigmoid_gate")
 
 
 def scaled_sum(a: torch.Tensor, scale_a: float, b: torch.Tensor, scale_b: float, out: torch.Tensor) -> None:
@@ -810,6 +829,49 @@ def diff_attention_mma(
         launch(ctx.decode_rows, ctx.decode_tokens, ctx.num_decode_rows, 1)
 
 
+SOFTCAP_NEAR_LIMIT = 0.45  # largest |score * scale / cap| that the four coefficients of the near form cover to 2e-7
+
+
+class SoftCap(ctypes.Structure):
+    """A soft cap on attention scores, ``cap * tanh(scale * raw / cap)``, as the tensor-core kernels take it
+    (csrc/softcap.cuh: KbSoftcap).  ``largest``: a bound on |raw| (the length of a query times that of a key) where one
+    is known: a small enough one lets the kernels use tanh(x) = x p(x^2) with the polynomial fitted here."""
+
+    _fields_ = [("mode", c_int), ("a", c_float), ("b", c_float), ("c", c_float * 4)]
+
+    @classmethod
+    def make(cls, scale: float, cap: float, largest: Optional[float] = None) -> "SoftCap":
+        if not (cap > 0.0 and scale > 0.0):
+            raise ValueError(f"a soft cap needs a positive cap and scale, got {cap!r} and {scale!r}")
+        log2e = math.log2(math.e)
+        held = cls(2, 2.0 * scale / cap * log2e, cap * log2e)
+        span = abs(scale) / cap * largest if largest is not None else math.inf
+        if span <= SOFTCAP_NEAR_LIMIT:
+            held.mode = 1
+            # tanh(x) / x as a cubic in z = x^2, interpolated at the four Chebyshev points of [0, span^2]
+            nodes = [0.5 * span * span * (1.0 + math.cos(math.pi * (2 * k + 1) / 8.0)) for k in range(4)]
+            values = [math.tanh(math.sqrt(z)) / math.sqrt(z) for z in nodes]
+            for i in range(1, 4):  # divided differences in place, then Newton's form multiplied out
+                for k in range(3, i - 1, -1):
+                    values[k] = (values[k] - values[k - 1]) / (nodes[k] - nodes[k - i])
+            p = [0.0, 0.0, 0.0, 0.0]
+            for k in range(3, -1, -1):
+                p = [(p[j - 1] if j else 0.0) - nodes[k] * p[j] for j in range(4)]
+                p[0] += values[k]
+            per = scale / cap  # x = raw * per; the result is raw * sum_j c_j raw^(2j)
+            for j in range(4):
+                held.c[j] = cap * log2e * p[j] * per ** (2 * j + 1)
+        return held
+
+    @property
+    def address(self) -> int:
+        return ctypes.addressof(self)
+
+
+def _softcap_address(softcap: Optional[SoftCap]) -> Optional[int]:
+    return softcap.address if softcap is not None else None
+
+
 ATTENTION_MMA_SINKS = True  # the tensor-core attention kernels take sink logits, in the step that divides a row's result
 
 DECODE_SPLIT = 128  # keys per split of the split-KV kernel (csrc/attention_mma.cu: DEC_SPLIT)
@@ -884,6 +946,7 @@ def attention_prefill_mma(
     two_tiles: Optional[bool] = None,
     sinks: Optional[torch.Tensor] = None,
     gate: Optional[torch.Tensor] = None,
+    softcap: Optional[SoftCap] = None,
 ) -> None:
     """Flash attention over query tiles (``attention_prefill_tile_rows`` queries each) of
     rows with several tokens (bf16).
@@ -899,7 +962,7 @@ def attention_prefill_mma(
 
     ``sinks``: fp32 [heads], a logit a head whose exp joins the softmax's denominator.  ``gate``: bf16 [tokens, >= heads *
     head_dim], columns laid out as ``out``'s; the result is multiplied by its sigmoid.  Every kernel here takes both, in its
-    last step (the tcgen05 kernels a gate whose rows are whole 16-byte groups)."""
+    last step (the tcgen05 kernels a gate whose rows are whole 16-byte groups).  ``softcap``: a cap on the scores."""
     what = "attention_prefill_mma"
     _need_cuda(what, q, out, k_cache, v_cache, qo_indptr, seq_lens, block_table, tile_rows, tile_starts, sinks, gate)
     _check_sinks(what, num_q_heads, sinks)
@@ -914,7 +977,7 @@ def attention_prefill_mma(
         fn = _fn(
             "attention_prefill_tc5",
             "kb_attention_prefill_tc5",
-            [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p],
         )
         merged = bool(_fn("attention_prefill_tc5", "kb_attention_prefill_tc5_merged", [c_int, c_int])(head_dim, page_size))
         splits = 1
@@ -947,7 +1010,7 @@ def attention_prefill_mma(
                 page_size, num_pages, float(scale), int(window), splits, _ptr(part_o), _ptr(part_ml),
                 wide_tiles[1].data_ptr() if use_two else None, wide_tiles[2].data_ptr() if use_two else None,
                 int(wide_tiles[0]) if use_two else 0, 1 if use_two else 0, _ptr(sinks), _ptr(gate), gate.stride(0) if gate is not None else 0,
-                _ptr(flag), _stream(),
+                _softcap_address(softcap), _ptr(flag), _stream(),
             ),
             what,
             launches=2 if splits > 1 else 1,
@@ -956,14 +1019,15 @@ def attention_prefill_mma(
     fn = _fn(
         "attention_mma",
         "kb_attention_prefill_mma",
-        [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+        [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p],
     )
     _check(
         fn(
             q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
             qo_indptr.data_ptr(), seq_lens.data_ptr(), block_table.data_ptr(), block_table.shape[1],
             tile_rows.data_ptr(), tile_starts.data_ptr(), int(num_tiles), num_q_heads, num_kv_heads, head_dim,
-            page_size, num_pages, float(scale), int(window), _ptr(sinks), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(flag), _stream(),
+            page_size, num_pages, float(scale), int(window), _ptr(sinks), _ptr(gate), gate.stride(0) if gate is not None else 0,
+            _softcap_address(softcap), _ptr(flag), _stream(),
         ),
         what,
     )
@@ -989,12 +1053,13 @@ def attention_decode_mma(
     num_splits: Optional[int] = None,
     sinks: Optional[torch.Tensor] = None,
     gate: Optional[torch.Tensor] = None,
+    softcap: Optional[SoftCap] = None,
 ) -> None:
     """Split-KV attention of rows that carry one token (bf16), then the merge.
 
     ``sinks``: fp32 [heads], a logit a head whose exp joins the softmax's denominator.  ``gate``: bf16 [tokens, >= heads *
     head_dim]; the result is multiplied by its sigmoid.  Both act where a row's result is divided (the merge, or the TMA-fed
-    kernel itself when it runs one split).
+    kernel itself when it runs one split).  ``softcap``: a cap on the scores.
 
     ``max_seq_len`` bounds every row's length; it sizes the grid and the scratch
     (``workspace.flat`` gives persistent fp32 buffers).  ``num_splits`` overrides the
@@ -1020,7 +1085,7 @@ def attention_decode_mma(
         fn = _fn(
             "attention_decode_tma",
             "kb_attention_decode_tma",
-            [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+            [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p],
         )
         joined = _joined_cache_map(k_cache, v_cache)  # keys and values in one copy where the cache allows
         map_k = joined or _cache_map(k_cache, bands=True)
@@ -1031,7 +1096,7 @@ def attention_decode_mma(
                 seq_lens.data_ptr(), block_table.data_ptr(), block_table.shape[1], decode_rows.data_ptr(),
                 decode_tokens.data_ptr(), int(num_rows), num_q_heads, num_kv_heads, head_dim, page_size, num_pages,
                 float(scale), int(window), num_splits, part_o.data_ptr(), part_ml.data_ptr(), 1 if joined else 0, _ptr(sinks), _ptr(gate),
-                gate.stride(0) if gate is not None else 0, _ptr(flag), _stream(),
+                gate.stride(0) if gate is not None else 0, _softcap_address(softcap), _ptr(flag), _stream(),
             ),
             what,
             launches=_fn("attention_decode_tma", "kb_attention_decode_tma_launches", [c_int])(num_splits),
@@ -1043,7 +1108,7 @@ def attention_decode_mma(
     fn = _fn(
         "attention_mma",
         "kb_attention_decode_mma",
-        [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+        [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p],
     )
     _check(
         fn(
@@ -1051,7 +1116,7 @@ def attention_decode_mma(
             seq_lens.data_ptr(), block_table.data_ptr(), block_table.shape[1], decode_rows.data_ptr(),
             decode_tokens.data_ptr(), int(num_rows), num_q_heads, num_kv_heads, head_dim, page_size, num_pages,
             float(scale), int(window), num_splits, part_o.data_ptr(), part_ml.data_ptr(), _ptr(sinks), _ptr(gate),
-            gate.stride(0) if gate is not None else 0, _ptr(flag), _stream(),
+            gate.stride(0) if gate is not None else 0, _softcap_address(softcap), _ptr(flag), _stream(),
         ),
         what,
         launches=2,
@@ -1236,7 +1301,7 @@ def _gemm_skinny(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Ten
     fn = _fn(
         "gemm_skinny", "kb_gemm_skinny_fused",
         [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-         c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p],
+         c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p],
     )
     _check(
         fn(x.data_ptr(), x.stride(0), weight.data_ptr(), weight.stride(0), _ptr(bias), _ptr(out),
@@ -1244,6 +1309,7 @@ def _gemm_skinny(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Ten
            _ptr(scale_by.sumsq) if scale_by is not None else None, scale_by.sumsq.shape[0] if scale_by is not None else 0,
            scale_by.hidden if scale_by is not None else 0, float(scale_by.eps) if scale_by is not None else 0.0,
            fold.residual.data_ptr() if fold is not None else None, fold.residual.stride(0) if fold is not None else 0,
+           _ptr(fold.scale) if fold is not None else None,
            fold.weight.data_ptr() if fold is not None else None, 1 if fold is not None and fold.weight.dtype == torch.bfloat16 else 0,
            fold.values.data_ptr() if fold is not None else None, fold.values.stride(0) if fold is not None else 0,
            fold.sumsq.data_ptr() if fold is not None else None, _stream()),
@@ -1346,13 +1412,15 @@ class PreNormed:
 @dataclass
 class ResidualNorm:
     """What a product does with its result instead of writing it: add it to the fp32 ``residual`` in
-    place, and leave ``values`` and ``sumsq`` of a :class:`PreNormed` for the norm (weight, eps) that follows."""
+    place (times ``scale``, fp32, a factor a column, where that is given), and leave ``values`` and ``sumsq`` of a
+    :class:`PreNormed` for the norm (weight, eps) that follows."""
 
     residual: torch.Tensor
     weight: torch.Tensor
     eps: float
     values: torch.Tensor
     sumsq: torch.Tensor
+    scale: Optional[torch.Tensor] = None
 
     def result(self) -> PreNormed:
         return PreNormed(self.values, self.sumsq, self.residual.shape[1], self.eps)
@@ -1672,6 +1740,19 @@ class PendingSums:
 
 
 @dataclass
+class PendingScaled:
+    """What a block that scales its sub-layers' results column by column leaves for the norm that reads the stream next:
+    ``residual += scale * values`` is still to be done, and that norm's kernel does it on its way."""
+
+    values: torch.Tensor
+    scale: torch.Tensor  # fp32 [hidden]
+
+    @property
+    def shape(self) -> torch.Size:
+        return self.values.shape
+
+
+@dataclass
 class ResidualCopy:
     """What a block that norms its sub-layers' OUTPUTS hands to the block after it: the residual's
     rows in the activation dtype (the sub-layers read the stream itself, so the next one wants them
@@ -1900,13 +1981,14 @@ def latent_norm_write(
     )
 
 
-def heads_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> None:
+def heads_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *, gate: Optional[torch.Tensor] = None) -> None:
     """A product per head: ``out[t, h, :] = weight[h] @ x[t, h, :]``.  ``x`` [tokens, heads, K] and
     ``out`` [tokens, heads, N] may be views with any row and head stride (inner stride 1: a head's columns
     may be part of a wider run); ``weight`` is
     contiguous [heads, N, K].  bfloat16: the library's batched product (fp32 accumulation);
-    float32: this package's FMA product, one launch a head."""
-    _need_cuda("heads_linear", x, weight, out)
+    float32: this package's FMA product, one launch a head.  ``gate`` [tokens, heads * N] (a view into wider rows is fine): the
+    result is multiplied by its sigmoid; ``out`` is then contiguous."""
+    _need_cuda("heads_linear", x, weight, out, gate)
     T, H, K = x.shape
     N = weight.shape[1]
     if weight.shape != (H, N, K) or out.shape != (T, H, N) or not weight.is_contiguous():
@@ -1922,10 +2004,14 @@ def heads_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> No
         for h in range(H):
             _check(fn(x.data_ptr() + 4 * h * x.stride(1), x.stride(0), weight.data_ptr() + 4 * h * N * K, K, None, out.data_ptr() + 4 * h * out.stride(1),
                       out.stride(0), T, N, K, _stream()), "heads_linear")
+        if gate is not None:
+            sigmoid_gate(out.view(T, H * N), gate)
         return
     if x.dtype != torch.bfloat16 or weight.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise KernelError("heads_linear: bfloat16 or float32 throughout")
     torch.bmm(x.transpose(0, 1), weight.transpose(1, 2), out=out.transpose(0, 1))
+    if gate is not None:
+        sigmoid_gate(out.view(T, H * N), gate)
 
 
 # ----------------------------------------------------------------------------- gated delta rule
@@ -2126,6 +2212,72 @@ def ssm_gated_norm(y: torch.Tensor, x: torch.Tensor, skip: torch.Tensor, z: torc
     fn = _fn("ssm", "kb_ssm_gated_norm", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_float, c_int, c_int, c_int, c_void_p, c_int, c_void_p])
     _check(fn(y.data_ptr(), x.data_ptr(), skip.data_ptr(), z.data_ptr(), z.stride(0), _is_bf16(z, what), weight.data_ptr(), float(eps), heads, vdim,
               norm_groups, out.data_ptr(), T, _stream()), what)
+
+
+# ----------------------------------------------------------------------------- real-gated linear recurrent unit
+
+RGLRU_MAX_TAPS = 16
+RGLRU_SEGMENTS = 32  # warps that share a request's tokens in the walk (csrc/rglru.cu: RG_MAX_SEGMENTS)
+
+
+def _check_rglru(what: str, x: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, rings: Optional[torch.Tensor], gate_bias: torch.Tensor,
+                 rate: torch.Tensor, parts: int) -> tuple[int, int, int]:
+    T, W = x.shape
+    n_taps = taps.shape[0]
+    if W % parts or x.stride(1) != 1:
+        raise KernelError(f"{what}: {W} columns with unit inner stride in {parts} equal parts")
+    for tensor, count in ((taps, n_taps * W), (conv_bias, W), (gate_bias, 2 * W), (rate, W)):
+        if tensor.dtype != torch.float32 or not tensor.is_contiguous() or tensor.numel() != count:
+            raise KernelError(f"{what}: taps [n, width], biases and rates are contiguous fp32 of the width's size")
+    if not 1 <= n_taps <= RGLRU_MAX_TAPS:
+        raise KernelError(f"{what}: {n_taps} taps (1 to {RGLRU_MAX_TAPS})")
+    if n_taps > 1 and (rings is None or rings.dtype != torch.float32 or not rings.is_contiguous() or tuple(rings.shape[1:]) != (n_taps, W)):
+        raise KernelError(f"{what}: the kept inputs must be contiguous fp32 [slots, taps, width]")
+    return T, W, n_taps
+
+
+def rglru_gates(x: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, rings: Optional[torch.Tensor], weights_t: torch.Tensor,
+                gate_bias: torch.Tensor, rate: torch.Tensor, a: torch.Tensor, into: torch.Tensor, *, row_ids: torch.Tensor, qo_indptr: torch.Tensor,
+                positions: torch.Tensor, state_slots: torch.Tensor, flag: Optional[torch.Tensor] = None) -> None:
+    """Convolution of ``x`` [tokens, width] over time (``taps`` [n, width] oldest first, earlier inputs from the requests' rings), the two
+    gates r and i (``weights_t`` [2, parts, n, n] as [gate, part, in, out], x's dtype; ``gate_bias`` [2, width]) and from them, per token and
+    channel in fp32, the decay ``a = exp(rate r)`` and the input term ``into = sqrt(1 - a^2) i u``."""
+    what = "rglru_gates"
+    _need_cuda(what, x, taps, conv_bias, rings, weights_t, gate_bias, rate, a, into, row_ids, qo_indptr, positions, state_slots, flag)
+    _need_i32(what, row_ids, qo_indptr, positions, state_slots)
+    parts = weights_t.shape[1]
+    T, W, n_taps = _check_rglru(what, x, taps, conv_bias, rings, gate_bias, rate, parts)
+    n = W // parts
+    if weights_t.shape != (2, parts, n, n) or weights_t.dtype != x.dtype or not weights_t.is_contiguous():
+        raise KernelError(f"{what}: the gates' matrices must be contiguous [2, parts, n, n] in x's dtype")
+    for tensor in (a, into):
+        if tensor.dtype != torch.float32 or tensor.shape != (T, W) or not tensor.is_contiguous():
+            raise KernelError(f"{what}: the outputs are contiguous fp32 [tokens, width]")
+    fn = _fn("rglru", "kb_rglru_gates", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int] + [c_void_p] * 8 + [c_int, c_int, c_void_p, c_void_p, c_int, c_int,
+                                                                                                               c_void_p, c_void_p])
+    _check(fn(x.data_ptr(), x.stride(0), _is_bf16(x, what), taps.data_ptr(), conv_bias.data_ptr(), n_taps, _ptr(rings), row_ids.data_ptr(), qo_indptr.data_ptr(),
+              positions.data_ptr(), state_slots.data_ptr(), weights_t.data_ptr(), gate_bias.data_ptr(), rate.data_ptr(), parts, n, a.data_ptr(),
+              into.data_ptr(), qo_indptr.numel() - 1, T, _ptr(flag), _stream()), what)
+
+
+def rglru_scan(a: torch.Tensor, into: torch.Tensor, x: torch.Tensor, y: torch.Tensor, states: torch.Tensor, rings: Optional[torch.Tensor], n_taps: int,
+               out: torch.Tensor, *, qo_indptr: torch.Tensor, positions: torch.Tensor, state_slots: torch.Tensor, segments: int = RGLRU_SEGMENTS) -> None:
+    """Every row's tokens in order through S <- a S + into, ``out = S gelu(y)`` (tanh form); ``states`` [slots, width] fp32 and the rings of kept
+    inputs [slots, taps, width] are left updated.  ``x`` and ``y``: the two branches' columns of the packed projection.  ``segments``: warps
+    that share a row's tokens (1: the plain walk, whose rounding does not depend on how a prompt was cut)."""
+    what = "rglru_scan"
+    _need_cuda(what, a, into, x, y, states, rings, out, qo_indptr, positions, state_slots)
+    _need_i32(what, qo_indptr, positions, state_slots)
+    T, W = a.shape
+    for tensor in (a, into, states) + ((rings,) if rings is not None else ()):
+        if tensor.dtype != torch.float32 or not tensor.is_contiguous():
+            raise KernelError(f"{what}: decays, input terms, states and rings are contiguous fp32")
+    if into.shape != a.shape or x.shape != a.shape or y.shape != a.shape or x.stride() != y.stride() or x.stride(1) != 1 or x.dtype != y.dtype or out.dtype != x.dtype \
+            or out.shape != a.shape or not out.is_contiguous() or states.shape[1:] != (W,) or (n_taps > 1 and (rings is None or tuple(rings.shape[1:]) != (n_taps, W))):
+        raise KernelError(f"{what}: shape or dtype mismatch")
+    fn = _fn("rglru", "kb_rglru_scan", [c_void_p] * 4 + [c_int] * 4 + [c_void_p] * 6 + [c_int, c_int, c_void_p])
+    _check(fn(a.data_ptr(), into.data_ptr(), x.data_ptr(), y.data_ptr(), x.stride(0), _is_bf16(x, what), W, int(n_taps), states.data_ptr(), _ptr(rings),
+              qo_indptr.data_ptr(), positions.data_ptr(), state_slots.data_ptr(), out.data_ptr(), qo_indptr.numel() - 1, int(segments), _stream()), what)
 
 
 # ----------------------------------------------------------------------------- mixture of experts

@@ -51,6 +51,7 @@ LIBRARIES: dict[str, list[str]] = {
     "projection_rope": [],
     "delta_rule": [],
     "ssm": [],
+    "rglru": [],
     "moe": [],
 }
 

@@ -64,6 +64,7 @@ def run_paged_attention(
     sinks: Optional[torch.Tensor] = None,
     value_dim: Optional[int] = None,
     gate: Optional[torch.Tensor] = None,
+    softcap: Optional["kernels.SoftCap"] = None,
 ) -> None:
     """Attention of every token of the step; picks the kernels for the dtype.
 
@@ -71,6 +72,7 @@ def run_paged_attention(
     is the first ``value_dim`` columns of its row (for a cache whose rows serve as keys and values);
     ``out`` keeps ``head_dim`` columns a head either way, of which the first ``value_dim`` are the result.
     ``gate`` ([tokens, heads * head_dim], the tensor-core kernels only): the result is multiplied by its sigmoid.
+    ``softcap`` (the tensor-core kernels only): a cap on the scores, the scale in it.
 
     float32: the fp32 kernel for all tokens (its arithmetic per token does not
     depend on the batch).  bfloat16: tensor-core kernels, query tiles for
@@ -85,8 +87,8 @@ def run_paged_attention(
         and (sinks is None or kernels.ATTENTION_MMA_SINKS)
     )
     if not use_mma:
-        if gate is not None:
-            raise ValueError("run_paged_attention: the 32-bit-arithmetic kernel takes no gate")
+        if gate is not None or softcap is not None:
+            raise ValueError("run_paged_attention: the 32-bit-arithmetic kernel takes neither gate nor cap")
         kernels.paged_attention_generic(
             qkv,
             out,
@@ -135,6 +137,7 @@ def run_paged_attention(
             wide_tiles=ctx.tiles.get(kernels.attention_prefill_wide_tile_rows(head_dim)),
             sinks=sinks,
             gate=gate,
+            softcap=softcap,
         )
     if ctx.num_decode_rows:
         with torch.cuda.stream(beside.stream) if beside is not None else contextlib.nullcontext():
@@ -156,6 +159,7 @@ def run_paged_attention(
                 flag=ctx.error_flag,
                 sinks=sinks,
                 gate=gate,
+                softcap=softcap,
             )
             if beside is not None:
                 beside.join.record()

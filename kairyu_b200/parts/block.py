@@ -33,6 +33,10 @@ class PreNormBlock(Block):
     (``kernels.ResidualNorm``), the product after it scales by the root mean square
     (``kernels.PreNormed``).  That needs norms that offer ``fold_target`` (RMSNorm does) and a
     mixer and feed-forward that offer ``fusable_norm``; any other part gets the plain flow.
+
+    ``LayerSpec.options["scale_names"]`` (two tensors, a factor a column each): the sub-layers' outputs are scaled by them
+    as they are added, ``x += s1 * mixer(norm(x)); x += s2 * ffn(norm(x))``; the scaling rides in whichever kernel adds
+    (``kernels.PendingScaled``, ``ResidualNorm.scale``), in 32-bit.  A layer may have no feed-forward.
     """
 
     graph_safe = True
@@ -47,25 +51,38 @@ class PreNormBlock(Block):
         self.ffn_norm = NORMS.build(layer.ffn_norm, **context) if layer.ffn is not None else None
         self.ffn = FEED_FORWARDS.build(layer.ffn, **context) if layer.ffn is not None else None
         self._parts = tuple(part for part in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if part is not None)
+        names = layer.options.get("scale_names")
+        self.scale_names = tuple(names)[: 1 if self.ffn is None else 2] if names is not None else ()
+        self.size = int(layer.mixer_norm.params["size"]) if self.scale_names else 0
+        self._scales: list[Optional[torch.Tensor]] = [None, None]  # fp32: they enter the residual sum
 
     def tensor_specs(self) -> list[TensorSpec]:
-        return [spec for part in self._parts for spec in part.tensor_specs()]
+        scales = [TensorSpec(name, (self.size,), role="vector", init="norm") for name in self.scale_names]
+        return [spec for part in self._parts for spec in part.tensor_specs()] + scales
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         for part in self._parts:
             part.load(tensors)
+        for index, name in enumerate(self.scale_names):
+            self._scales[index] = tensors[name].float().contiguous()
 
     def bytes_streamed(self) -> int:
-        return sum(part.bytes_streamed() for part in self._parts)
+        return sum(part.bytes_streamed() for part in self._parts) + sum(4 * s.numel() for s in self._scales if s is not None)
+
+    def _pending(self, index: int, output: torch.Tensor):
+        return output if self._scales[index] is None else kernels.PendingScaled(output, self._scales[index])
 
     def _fused(self, ctx: StepContext) -> bool:
-        if ctx.dtype != torch.bfloat16 or self.ffn is None or not kernels.fused_norm_available():
+        if ctx.dtype != torch.bfloat16 or not kernels.fused_norm_available():
             return False
-        if not (hasattr(self.mixer_norm, "fold_target") and hasattr(self.ffn_norm, "fold_target")):
-            return False  # a norm offers ``fold_target`` when the products around it can take its two halves
-        mixer_ok = getattr(self.mixer, "fusable_norm", None)
-        ffn_ok = getattr(self.ffn, "fusable_norm", None)
-        return bool(mixer_ok and ffn_ok and mixer_ok(ctx.num_tokens) and ffn_ok(ctx.num_tokens))
+        # a norm offers ``fold_target`` when the products around it can take its two halves
+        for norm, part in ((self.mixer_norm, self.mixer), (self.ffn_norm, self.ffn)):
+            if part is None:
+                continue
+            fusable = getattr(part, "fusable_norm", None)
+            if not hasattr(norm, "fold_target") or fusable is None or not fusable(ctx.num_tokens):
+                return False
+        return True
 
     def prenorm_target(self, ctx: StepContext) -> Optional[Norm]:
         """The norm the block before this one may fold into its last product, or None."""
@@ -83,15 +100,21 @@ class PreNormBlock(Block):
             normed = delta
         else:
             normed = self.mixer_norm.apply(residual, delta, ctx)
+        fused = self._fused(ctx)
         if self.ffn is None:
-            return residual, self.mixer.forward(normed, ctx, cache)
-        if not self._fused(ctx):
+            if not fused or next_norm is None:
+                return residual, self._pending(0, self.mixer.forward(normed, ctx, cache))
+            # (its own input may lie in the same buffer: the products that read it are done when the last one writes)
+            fold = next_norm.fold_target(residual, ctx, "mixer", self._scales[0])
+            return residual, self.mixer.forward(normed, ctx, cache, fold=fold)
+        if not fused:
             mixed = self.mixer.forward(normed, ctx, cache)
-            normed = self.ffn_norm.apply(residual, mixed, ctx)
-            return residual, self.ffn.forward(normed, ctx)
-        mixed = self.mixer.forward(normed, ctx, cache, fold=self.ffn_norm.fold_target(residual, ctx, "ffn"))
-        fold = next_norm.fold_target(residual, ctx, "mixer") if next_norm is not None else None
-        return residual, self.ffn.forward(mixed, ctx, fold=fold)
+            normed = self.ffn_norm.apply(residual, self._pending(0, mixed), ctx)
+            return residual, self._pending(1, self.ffn.forward(normed, ctx))
+        mixed = self.mixer.forward(normed, ctx, cache, fold=self.ffn_norm.fold_target(residual, ctx, "ffn", self._scales[0]))
+        fold = next_norm.fold_target(residual, ctx, "mixer", self._scales[1]) if next_norm is not None else None
+        output = self.ffn.forward(mixed, ctx, fold=fold)
+        return residual, output if fold is not None else self._pending(1, output)
 
 
 @BLOCKS.register("output_norm")

@@ -17,6 +17,10 @@ what a query sees of a value depends on their distance alone.  ``own_kv=False``:
 (nor their norm); it attends over a cache that another layer's call wrote in the same step, with queries, sink and gate of
 its own (the run order names that slot with ``writes_cache=False``).
 
+``qk_norm="turned"``: every head of q and k is divided by its root mean square BEHIND its rotation, without a weight.
+``values="keys"``: there is no value projection; a value is the key as projected, before norm and rotation (``value_dim ==
+head_dim``).  ``softcap``: scores become ``softcap * tanh(scale * q.k / softcap)`` before the softmax.
+
 ``sink``: ``None`` (a plain softmax), ``"zero"`` (a sink of logit 0: one added to the denominator, no tensor) or
 ``"learned"`` (tensor ``<prefix>.sink``, one logit a query head).  A sink is a term exp(sink) of the denominator alone, taken as stored.
 The gate reads the mixer's input, as the projections do.  Query head h uses key/value head
@@ -26,7 +30,7 @@ bfloat16 with ``head_dim == value_dim`` of a size the paged tensor-core kernels 
 tiles, single tokens split over the keys), the sink in their last step and the gate at their store; everything else runs the
 32-bit-arithmetic kernel.
 
-Tensors under ``prefix``: ``q``, ``k``, ``v``, ``o``, and ``g``, ``q.norm``, ``k.norm``, ``sink`` as the options ask.
+Tensors under ``prefix``: ``q``, ``k``, ``v`` (unless values are keys), ``o``, and ``g``, ``q.norm``, ``k.norm``, ``sink`` as the options ask.
 """
 
 from __future__ import annotations
@@ -63,6 +67,8 @@ class GatedAttention(Mixer):
         window: Optional[int] = None,
         value_position: Optional[PartSpec] = None,
         own_kv: bool = True,
+        values: str = "projected",
+        softcap: Optional[float] = None,
         dtype: torch.dtype,
         device: str,
         shared: Optional[dict] = None,
@@ -70,8 +76,10 @@ class GatedAttention(Mixer):
     ) -> None:
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads are not a multiple of {num_kv_heads} KV heads")
-        if qk_norm not in (None, "projection", "head"):
-            raise ValueError(f"unknown query/key norm {qk_norm!r} (None, 'projection', 'head')")
+        if qk_norm not in (None, "projection", "head", "turned"):
+            raise ValueError(f"unknown query/key norm {qk_norm!r} (None, 'projection', 'head', 'turned')")
+        if values not in ("projected", "keys") or (values == "keys" and (value_dim != head_dim or value_position is not None)):
+            raise ValueError("values are 'projected', or 'keys' of the keys' width that do not turn")
         if sink not in (None, "zero", "learned"):
             raise ValueError(f"unknown sink {sink!r} (None, 'zero', 'learned')")
         self.prefix = prefix
@@ -90,6 +98,11 @@ class GatedAttention(Mixer):
         self.dtype = dtype
         self.device = device
         self.own_kv = bool(own_kv)
+        self.keys_are_values = values == "keys"
+        self.softcap = float(softcap) if softcap is not None else None
+        # a head of unit mean square is sqrt(head_dim) long, give or take its rounding to the activations' dtype
+        longest = 1.01 * head_dim if qk_norm == "turned" else None
+        self.cap = kernels.SoftCap.make(self.scale, self.softcap, longest) if softcap is not None else None
         table = shared if shared is not None else {}
 
         def encoding(spec: Optional[PartSpec], width: int):
@@ -106,11 +119,11 @@ class GatedAttention(Mixer):
         self.value_position = encoding(value_position, value_dim)
         self.q_size = num_heads * head_dim
         self.k_size = num_kv_heads * head_dim if self.own_kv else 0
-        self.v_size = num_kv_heads * value_dim if self.own_kv else 0
+        self.v_size = num_kv_heads * value_dim if self.own_kv and not self.keys_are_values else 0
         self.out_size = num_heads * value_dim
         self.k_offset = self.q_size
-        self.v_offset = self.q_size + self.k_size
-        self.g_offset = self.v_offset + self.v_size
+        self.v_offset = self.k_offset if self.keys_are_values else self.q_size + self.k_size
+        self.g_offset = self.q_size + self.k_size + self.v_size
         self.packed_width = self.g_offset + (self.out_size if gate else 0)
         self.w_in: Optional[torch.Tensor] = None  # [q | k | v | g rows, hidden]
         self.w_o: Optional[torch.Tensor] = None
@@ -123,8 +136,10 @@ class GatedAttention(Mixer):
         p = self.prefix
         specs = [TensorSpec(f"{p}.q", (self.q_size, self.hidden_size))]
         if self.own_kv:
-            specs += [TensorSpec(f"{p}.k", (self.k_size, self.hidden_size)), TensorSpec(f"{p}.v", (self.v_size, self.hidden_size))]
-        if self.qk_norm:
+            specs.append(TensorSpec(f"{p}.k", (self.k_size, self.hidden_size)))
+            if not self.keys_are_values:
+                specs.append(TensorSpec(f"{p}.v", (self.v_size, self.hidden_size)))
+        if self.qk_norm in ("projection", "head"):
             per_head = self.qk_norm == "head"
             specs.append(TensorSpec(f"{p}.q.norm", (self.head_dim if per_head else self.q_size,), role="vector", init="norm"))
             if self.own_kv:
@@ -138,10 +153,14 @@ class GatedAttention(Mixer):
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         p = self.prefix
-        rows = [tensors[f"{p}.q"]] + ([tensors[f"{p}.k"], tensors[f"{p}.v"]] if self.own_kv else []) + ([tensors[f"{p}.g"]] if self.gate else [])
+        rows = [tensors[f"{p}.q"]]
+        if self.own_kv:
+            rows += [tensors[f"{p}.k"]] + ([] if self.keys_are_values else [tensors[f"{p}.v"]])
+        if self.gate:
+            rows.append(tensors[f"{p}.g"])
         self.w_in = torch.cat(rows, dim=0).contiguous()
         self.w_o = tensors[f"{p}.o"].contiguous()
-        if self.qk_norm:
+        if self.qk_norm in ("projection", "head"):
             self.q_norm_weight = tensors[f"{p}.q.norm"].contiguous()
             # without keys of its own the kernel norms no key; it still wants the two weights as a pair
             self.k_norm_weight = tensors[f"{p}.k.norm"].contiguous() if self.own_kv else self.q_norm_weight
@@ -175,7 +194,13 @@ class GatedAttention(Mixer):
         return (kernels.attention_prefill_tile_rows(self.head_dim),) + ((wide,) if wide else ())
 
     # -- compute
-    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
+    def fusable_norm(self, tokens: int) -> bool:
+        """Whether the input and the output product can take the norms around them into their epilogues."""
+        return kernels.fused_norm_shapes_ok(tokens, self.hidden_size, self.out_size)
+
+    def forward(self, x, ctx: StepContext, cache: CacheView, fold=None):
+        """``x``: rows, or a ``kernels.PreNormed``; ``fold`` (a ``kernels.ResidualNorm``): the output
+        product adds its result to the residual and returns the ``PreNormed`` for the next norm."""
         tokens = x.shape[0]
         ws = ctx.workspace
         packed = ws.buffer("gattn.packed", tokens, self.packed_width, self.dtype)
@@ -192,23 +217,26 @@ class GatedAttention(Mixer):
             q_norm_weight=self.q_norm_weight, k_norm_weight=self.k_norm_weight, eps=self.norm_eps, cos=cos, sin=sin,
             interleaved=self.rotary_interleaved, block_table=block_table if writes else None,
             write_from=ctx.write_from if writes else None, k_cache=cache.k if writes else None, v_cache=cache.v if writes else None,
-            flag=ctx.error_flag, per_head_norm=self.qk_norm == "head", v_cos=v_cos if writes else None, v_sin=v_sin if writes else None,
+            flag=ctx.error_flag, per_head_norm=self.qk_norm == "head", unit_heads=self.qk_norm == "turned", v_cos=v_cos if writes else None, v_sin=v_sin if writes else None,
         )
         mixed = ws.buffer("gattn.mixed", tokens, self.out_size, self.dtype)
         gate = packed[:, self.g_offset :] if self.gate else None
         if self._tensor_cores() and not ctx.extras.get("force_generic_attention", False):
             run_paged_attention(packed, mixed, cache, ctx, num_q_heads=self.num_heads, num_kv_heads=self.num_kv_heads, head_dim=self.head_dim,
-                                scale=self.scale, window=self.window or 0, sinks=self.sinks, gate=gate)
+                                scale=self.scale, window=self.window or 0, sinks=self.sinks, gate=gate, softcap=self.cap)
         else:
             kernels.diff_attention_generic(
                 packed, mixed, cache.k, cache.v, positions=ctx.positions, row_ids=ctx.row_ids, block_table=block_table,
-                num_q_heads=self.num_heads, maps=1, scale=self.scale, window=self.window or 0, sinks=self.sinks, gate=gate, flag=ctx.error_flag,
+                num_q_heads=self.num_heads, maps=1, scale=self.scale, softcap=self.softcap or 0.0, window=self.window or 0, sinks=self.sinks, gate=gate, flag=ctx.error_flag,
             )
         if v_cos is not None:  # the values were cached turned by their positions: turn each head's sum back by the query's
             if self.gate:
                 raise ValueError("turned values with an output gate: the gate would have to follow the turning back")
             kernels.rotate_heads(mixed, heads=self.num_heads, head_dim=self.value_dim, cos=v_cos, sin=v_sin, positions=ctx.positions,
                                  interleaved=self.rotary_interleaved, inverse=True, flag=ctx.error_flag)
+        if fold is not None:
+            kernels.linear(mixed, self.w_o, None, None, fold=fold)
+            return fold.result()
         out = ws.buffer("gattn.out", tokens, self.hidden_size, self.dtype)
         kernels.linear(mixed, self.w_o, None, out)
         return out

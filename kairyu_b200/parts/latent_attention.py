@@ -18,6 +18,9 @@ behind the latent row, the rotated query part stands behind the query carried in
 the attention kernels see one key/value head of width ``kv_rank + rot_dim`` whose values are the first
 ``kv_rank`` columns of its rows.
 
+``gate``: the heads' results side by side are multiplied by ``sigmoid(W_g x)`` (tensor ``<prefix>.g``; its rows ride in the input
+product) before the output product.
+
 ``sink``: a learned logit a head (tensor ``<prefix>.sink``) that joins the softmax's denominator and
 nothing else (exp(sink) is one more term of the sum, taken as stored: no row of the cache stands behind it).
 """
@@ -53,6 +56,7 @@ class LatentAttention(Mixer):
         position: Optional[PartSpec] = None,
         rotary_interleaved: bool = True,
         sink: bool = False,
+        gate: bool = False,
         dtype: torch.dtype,
         device: str,
         shared: Optional[dict] = None,
@@ -72,6 +76,7 @@ class LatentAttention(Mixer):
             if self.position.rotary_dim != rot_dim:
                 raise ValueError(f"the rotary encoding turns {self.position.rotary_dim} dimensions, the rotated part has {rot_dim}")
         self.has_sink = sink
+        self.gate = bool(gate)
         self.sinks: Optional[torch.Tensor] = None
         self.prefix = prefix
         self.hidden_size = hidden_size
@@ -86,7 +91,9 @@ class LatentAttention(Mixer):
         self.q_head_width = head_dim + rot_dim
         self.q_size = num_heads * self.q_head_width
         self.row_width = kv_rank + rot_dim  # a cached row: the latent, then the rotated key part
-        self.w_in: Optional[torch.Tensor] = None      # [q_size + kv_rank, hidden]: q rows, then the down-projection's
+        self.out_size = num_heads * value_dim
+        self.packed_width = self.q_size + self.row_width + (self.out_size if self.gate else 0)
+        self.w_in: Optional[torch.Tensor] = None      # q rows, then the down-projection's, then the gate's
         self.latent_norm: Optional[torch.Tensor] = None
         self.w_absorb: Optional[torch.Tensor] = None  # [heads, kv_rank, head_dim]: W_uk[h]^T
         self.w_up_v: Optional[torch.Tensor] = None    # [heads, value_dim, kv_rank]
@@ -101,11 +108,13 @@ class LatentAttention(Mixer):
             TensorSpec(f"{p}.uk", (self.num_heads * self.head_dim, self.kv_rank)),
             TensorSpec(f"{p}.uv", (self.num_heads * self.value_dim, self.kv_rank)),
             TensorSpec(f"{p}.o", (self.hidden_size, self.num_heads * self.value_dim)),
-        ] + ([TensorSpec(f"{p}.sink", (self.num_heads,), role="vector", init="normal")] if self.has_sink else [])
+        ] + ([TensorSpec(f"{p}.g", (self.out_size, self.hidden_size))] if self.gate else []) \
+            + ([TensorSpec(f"{p}.sink", (self.num_heads,), role="vector", init="normal")] if self.has_sink else [])
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         p = self.prefix
-        self.w_in = torch.cat([tensors[f"{p}.q"], tensors[f"{p}.dkv"]], dim=0).contiguous()
+        rows = [tensors[f"{p}.q"], tensors[f"{p}.dkv"]] + ([tensors[f"{p}.g"]] if self.gate else [])
+        self.w_in = torch.cat(rows, dim=0).contiguous()
         self.latent_norm = tensors[f"{p}.dkv.norm"].contiguous()
         self.w_absorb = tensors[f"{p}.uk"].view(self.num_heads, self.head_dim, self.kv_rank).transpose(1, 2).contiguous()
         self.w_up_v = tensors[f"{p}.uv"].view(self.num_heads, self.value_dim, self.kv_rank).contiguous()
@@ -132,11 +141,17 @@ class LatentAttention(Mixer):
         wide = kernels.attention_prefill_wide_tile_rows(self.row_width)
         return (kernels.attention_prefill_tile_rows(self.row_width),) + ((wide,) if wide else ())
 
-    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
+    def fusable_norm(self, tokens: int) -> bool:
+        """Whether the input and the output product can take the norms around them into their epilogues."""
+        return kernels.fused_norm_shapes_ok(tokens, self.hidden_size, self.out_size)
+
+    def forward(self, x, ctx: StepContext, cache: CacheView, fold=None):
+        """``x``: rows, or a ``kernels.PreNormed``; ``fold`` (a ``kernels.ResidualNorm``): the output
+        product adds its result to the residual and returns the ``PreNormed`` for the next norm."""
         tokens = x.shape[0]
         ws = ctx.workspace
         heads, rank, width = self.num_heads, self.kv_rank, self.row_width
-        packed = ws.buffer("latent.packed", tokens, self.q_size + width, self.dtype)
+        packed = ws.buffer("latent.packed", tokens, self.packed_width, self.dtype)
         kernels.linear(x, self.w_in, None, packed)
         # a query row a head: [the query carried into the latent space | its rotated part], as wide as a cached row
         q_latent = ws.buffer("latent.q", tokens, heads * width, self.dtype)
@@ -163,8 +178,12 @@ class LatentAttention(Mixer):
             run_paged_attention(q_latent[:, columns], mixed[:, columns], rows, ctx, num_q_heads=count, num_kv_heads=1, head_dim=width,
                                 scale=self.scale, window=self.window or 0, value_dim=rank,
                                 sinks=self.sinks[first : first + count] if self.sinks is not None else None)
-        values = ws.buffer("latent.values", tokens, heads * self.value_dim, self.dtype)
-        kernels.heads_linear(mixed.view(tokens, heads, width)[:, :, :rank], self.w_up_v, values.view(tokens, heads, self.value_dim))
+        values = ws.buffer("latent.values", tokens, self.out_size, self.dtype)
+        kernels.heads_linear(mixed.view(tokens, heads, width)[:, :, :rank], self.w_up_v, values.view(tokens, heads, self.value_dim),
+                             gate=packed[:, self.q_size + width :] if self.gate else None)
+        if fold is not None:
+            kernels.linear(values, self.w_o, None, None, fold=fold)
+            return fold.result()
         out = ws.buffer("latent.out", tokens, self.hidden_size, self.dtype)
         kernels.linear(values, self.w_o, None, out)
         return out

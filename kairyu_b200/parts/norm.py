@@ -65,7 +65,10 @@ class RMSNorm(Norm):
         if isinstance(delta, kernels.PendingGated):  # a gated sub-layer output still to be added
             kernels.gated_residual_norm(residual, delta, self.weight, self.eps, out, rows=rows)
             return out
-        kernels.rmsnorm(residual, self.weight, self.eps, out, delta=delta, rows=rows)
+        scale = None
+        if isinstance(delta, kernels.PendingScaled):  # a sub-layer output that is scaled column by column as it is added
+            delta, scale = delta.values, delta.scale
+        kernels.rmsnorm(residual, self.weight, self.eps, out, delta=delta, delta_scale=scale, rows=rows)
         return out
 
     def pending(self, y: torch.Tensor) -> "kernels.PendingNormed":
@@ -84,14 +87,15 @@ class RMSNorm(Norm):
         kernels.output_norm_add(residual, y, self.weight, self.eps, copy)
         return residual if copy is None else copy
 
-    def fold_target(self, residual: torch.Tensor, ctx: StepContext, tag: str) -> "kernels.ResidualNorm":
+    def fold_target(self, residual: torch.Tensor, ctx: StepContext, tag: str, scale: Optional[torch.Tensor] = None) -> "kernels.ResidualNorm":
         """For a product that takes this norm's first half into its epilogue: it adds its result
         to ``residual`` and leaves the rows weighted and their sums of squares; the product that
-        reads them scales by the root mean square (kernels.ResidualNorm / kernels.PreNormed)."""
+        reads them scales by the root mean square (kernels.ResidualNorm / kernels.PreNormed).  ``scale``
+        (fp32, a factor a column): what is added is scaled by it."""
         rows = residual.shape[0]
         values = ctx.workspace.buffer(f"norm.fold.{tag}.values", rows, self.size, torch.bfloat16)
         sumsq = ctx.workspace.flat(f"norm.fold.{tag}.sumsq", 16 * kernels.skinny_blocks(rows, self.size), torch.float32).view(-1, 16)
-        return kernels.ResidualNorm(residual, self.weight, self.eps, values, sumsq)
+        return kernels.ResidualNorm(residual, self.weight, self.eps, values, sumsq, scale)
 
 
 @NORMS.register("layernorm")

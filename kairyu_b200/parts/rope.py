@@ -39,7 +39,7 @@ def _yarn_amplitude(factor: float, mscale: float = 1.0) -> float:
     return 1.0 + 0.1 * mscale * math.log(factor) if factor > 1.0 else 1.0
 
 
-def _yarn_inv_freq(dim: int, theta: float, scaling: RopeScaling) -> tuple[torch.Tensor, float]:
+def _yarn_inv_freq(dim: int, theta: float, scaling: RopeScaling, dtype: torch.dtype = torch.float32) -> tuple[torch.Tensor, float]:
     """Yarn ("NTK by parts"): pairs of the head that turn often within the original context keep
     their frequency, pairs that turn less than ``beta_slow`` times are slowed ``factor`` times
     (positions interpolated), and the pairs between blend the two linearly in the pair index.
@@ -47,7 +47,7 @@ def _yarn_inv_freq(dim: int, theta: float, scaling: RopeScaling) -> tuple[torch.
     original context L; solved for i, ``turns`` turns are made by pair
     dim * ln(L / (2 pi turns)) / (2 ln theta).  The blend's ends are that index for ``beta_fast``
     rounded down and for ``beta_slow`` rounded up, as kairyu/models/layers.py:55-81 has them."""
-    base = theta ** (torch.arange(0, dim, 2, dtype=torch.int64).float() / dim)
+    base = theta ** (torch.arange(0, dim, 2, dtype=torch.int64).to(dtype) / dim)
     kept, slowed = 1.0 / base, 1.0 / (scaling.factor * base)
     context = scaling.original_max_position_embeddings
 
@@ -56,12 +56,14 @@ def _yarn_inv_freq(dim: int, theta: float, scaling: RopeScaling) -> tuple[torch.
 
     first = max(math.floor(pair_with(scaling.beta_fast)), 0)
     last = min(math.ceil(pair_with(scaling.beta_slow)), dim - 1)
-    span = last - first if last != first else 0.001
-    slowed_share = ((torch.arange(dim // 2).float() - first) / span).clamp(0, 1)
+    span = max(last - first, 0.001)
+    slowed_share = ((torch.arange(dim // 2).to(dtype) - first) / span).clamp(0, 1)
     inv_freq = slowed * slowed_share + kept * (1.0 - slowed_share)
     amplitude = _yarn_amplitude(scaling.factor)
     if scaling.mscale is not None and scaling.mscale_all_dim is not None:
         amplitude = _yarn_amplitude(scaling.factor, scaling.mscale) / _yarn_amplitude(scaling.factor, scaling.mscale_all_dim)
+    if scaling.amplitude is not None:
+        amplitude = scaling.amplitude
     return inv_freq, amplitude
 
 
@@ -70,17 +72,18 @@ def rotary_tables(
 ) -> tuple[torch.Tensor, torch.Tensor]:
     """(cos, sin), each [max_positions, dim/2] fp32, on the CPU.  ``wide_angles``: frequencies theta^(-2i/dim) and
     angles position * frequency are formed in 64-bit and only cos and sin are rounded to 32-bit, so that an entry
-    is the correctly rounded value at every position (no scaling, or the llama3 or linear kind)."""
+    is the correctly rounded value at every position."""
     if wide_angles:
-        if scaling is not None and scaling.kind not in ("llama3", "linear"):
-            raise ValueError("wide angles come without frequency scaling, or with the llama3 or the linear kind")
+        factor = 1.0
         inv_freq = theta ** (-torch.arange(0, dim, 2, dtype=torch.float64) / dim)
         if scaling is not None and scaling.kind == "llama3":
             inv_freq = _llama3_inv_freq(inv_freq, scaling)
+        elif scaling is not None and scaling.kind == "yarn":
+            inv_freq, factor = _yarn_inv_freq(dim, theta, scaling, torch.float64)
         elif scaling is not None:
             inv_freq = inv_freq / scaling.factor
         freqs = torch.arange(max_positions, dtype=torch.float64)[:, None] * inv_freq[None, :]
-        return freqs.cos().float().contiguous(), freqs.sin().float().contiguous()
+        return (freqs.cos() * factor).float().contiguous(), (freqs.sin() * factor).float().contiguous()
     factor = 1.0
     if scaling is not None and scaling.kind == "yarn":
         inv_freq, factor = _yarn_inv_freq(dim, theta, scaling)

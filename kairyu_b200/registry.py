@@ -74,6 +74,9 @@ def _register_builtin() -> None:
     from kairyu_b200.models import koravik
 
     register_architecture("Koravik", koravik.parse_koravik, koravik.koravik_spec)
+    from kairyu_b200.models import rezelix
+
+    register_architecture("Rezelix", rezelix.parse_rezelix, rezelix.rezelix_spec)
 
 
 _register_builtin()

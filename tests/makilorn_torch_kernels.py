@@ -40,8 +40,11 @@ def latent_norm_write(packed, offset, rank, weight, eps, cache, *, positions, ro
         cache[page, position % page_size, 0] = c[t].to(cache.dtype)
 
 
-def heads_linear(x, weight, out):
-    out.copy_(torch.einsum("thk,hnk->thn", x.float(), weight.float()).to(out.dtype))
+def heads_linear(x, weight, out, *, gate=None):
+    y = torch.einsum("thk,hnk->thn", x.float(), weight.float())
+    if gate is not None:
+        y = y * torch.sigmoid(gate.float()).reshape(y.shape)
+    out.copy_(y.to(out.dtype))
 
 
 def _convolve(inputs_of_row, taps, conv_state, qo_indptr, state_slots, tokens, bias=None):

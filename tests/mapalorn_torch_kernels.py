@@ -55,7 +55,8 @@ def _place(cache, block_table, write_from, row, position):
 
 def projection_norm_rope_write(packed, *, num_q_heads, num_kv_heads, head_dim, value_dim, k_offset, v_offset, positions, row_ids,
                                q_norm_weight=None, k_norm_weight=None, eps=0.0, cos=None, sin=None, interleaved=False, block_table=None,
-                               write_from=None, k_cache=None, v_cache=None, flag=None, per_head_norm=False, v_cos=None, v_sin=None):
+                               write_from=None, k_cache=None, v_cache=None, flag=None, per_head_norm=False, unit_heads=False,
+                               v_cos=None, v_sin=None):
     q_size, k_size, v_size = num_q_heads * head_dim, num_kv_heads * head_dim, num_kv_heads * value_dim
     for t in range(packed.shape[0]):
         position, row = int(positions[t]), int(row_ids[t])
@@ -72,6 +73,9 @@ def projection_norm_rope_write(packed, *, num_q_heads, num_kv_heads, head_dim, v
                 q[h] = _turn(q[h], cos[position], sin[position], interleaved)
             for h in range(num_kv_heads):
                 k[h] = _turn(k[h], cos[position], sin[position], interleaved)
+        if unit_heads:
+            q = q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps)
+            k = k * torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + eps)
         packed[t, :q_size] = q.reshape(-1).to(packed.dtype)
         if k_cache is not None:
             place = _place(k_cache, block_table, write_from, row, position)

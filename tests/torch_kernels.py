@@ -26,7 +26,9 @@ def patch_tokens(ids, source, sampled, flag=None):
             ids[t] = sampled[int(source[t])]
 
 
-def rmsnorm(x, weight, eps, out, *, delta=None, rows=None):
+def rmsnorm(x, weight, eps, out, *, delta=None, delta_scale=None, rows=None):
+    if delta_scale is not None:
+        delta = delta.float() * delta_scale
     if rows is not None:
         v = x[rows.long()].float()
         if delta is not None:
