@@ -1,0 +1,64 @@
+// What the kernels of the real-gated linear recurrent unit share: the short convolution over a step's rows and a request's ring of
+// kept inputs, and the step from gate sums to a decay and an input term (rglru.cu says what is computed).
+#pragma once
+#include "common.cuh"
+
+#define RG_MAX_TAPS 16
+
+__device__ __forceinline__ float sigmoid_exact(float z) { return 1.0f / (1.0f + expf(-z)); }
+// the same by the fast exponential and quotient (2 ulp): for the bfloat16 mode's kernels
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
+__device__ __forceinline__ float sqrt_fast(float x) {
+    float y;
+    asm("sqrt.approx.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float gelu_tanh_f(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+
+// 1 - e^(-y) for y >= 0: the series of the exponential where the difference would cancel
+template <bool EXACT>
+__device__ __forceinline__ float one_minus_exp_neg(float y) {
+    float p = -1.0f / 40320.0f;
+    p = fmaf(p, y, 1.0f / 5040.0f);
+    p = fmaf(p, y, -1.0f / 720.0f);
+    p = fmaf(p, y, 1.0f / 120.0f);
+    p = fmaf(p, y, -1.0f / 24.0f);
+    p = fmaf(p, y, 1.0f / 6.0f);
+    p = fmaf(p, y, -0.5f);
+    p = fmaf(p, y, 1.0f);
+    return y < 0.35f ? p * y : 1.0f - (EXACT ? expf(-y) : __expf(-y));
+}
+
+// gate sums (biases added) and the convolved input of one channel -> the decay a and the input term
+template <bool EXACT>
+__device__ __forceinline__ void rglru_terms(float pre_r, float pre_i, float rate, float u, float& a, float& into) {
+    if (EXACT) {
+        const float la = rate * sigmoid_exact(pre_r);
+        a = expf(la);
+        into = sqrtf(one_minus_exp_neg<true>(-2.0f * la)) * sigmoid_exact(pre_i) * u;
+    } else {
+        const float la = rate * sigmoid_fast(pre_r);
+        a = __expf(la);
+        into = sqrt_fast(one_minus_exp_neg<false>(-2.0f * la)) * sigmoid_fast(pre_i) * u;
+    }
+}
+
+struct RglruConv {
+    const float* taps;  // [n_taps, W], oldest first
+    const float* bias;  // [W]
+    int n_taps, W;
+};
+
+// the convolved input of channel c of token t (position pos, offset o within its row's tokens); x: the step's rows of the
+// x branch; ring: the request's kept inputs
+template <typename T>
+__device__ __forceinline__ float rglru_conv(const T* __restrict__ x, int stride, const float* __restrict__ ring, const RglruConv& conv,
+                                            int t, int o, int pos, int c) {
+    float z = conv.bias[c];
+    for (int back = conv.n_taps - 1; back >= 0; --back) {
+        if (pos - back < 0) continue;  // zeros before the start
+        const float in = o - back >= 0 ? to_float(x[(size_t)(t - back) * stride + c]) : ring[(size_t)((pos - back) % conv.n_taps) * conv.W + c];
+        z = fmaf(conv.taps[(size_t)(conv.n_taps - 1 - back) * conv.W + c], in, z);
+    }
+    return z;
+}

@@ -2260,6 +2260,67 @@ def rglru_gates(x: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, ri
               into.data_ptr(), qo_indptr.numel() - 1, T, _ptr(flag), _stream()), what)
 
 
+def rglru_tc5_supported(part_width: int) -> bool:
+    """Part widths the tensor-core kernel of the gates takes (bfloat16): whole 16-byte groups."""
+    return part_width % 8 == 0
+
+
+def _check_rglru_padded(what: str, weights: torch.Tensor, n: int) -> int:
+    np = weights.shape[2]
+    if weights.dtype != torch.bfloat16 or weights.dim() != 4 or weights.shape[0] != 2 or weights.shape[3] != np or np % 16 or np < n or not weights.is_contiguous():
+        raise KernelError(f"{what}: the gates' matrices must be contiguous bfloat16 [2, parts, np, np], np the part's width rounded up to 16")
+    return np
+
+
+def rglru_gates_tc5(x: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, rings: Optional[torch.Tensor], weights: torch.Tensor,
+                    gate_bias: torch.Tensor, rate: torch.Tensor, a: torch.Tensor, into: torch.Tensor, *, row_ids: torch.Tensor, qo_indptr: torch.Tensor,
+                    positions: torch.Tensor, state_slots: torch.Tensor, flag: Optional[torch.Tensor] = None) -> None:
+    """``rglru_gates`` on tensor cores (bfloat16).  ``weights``: [2, parts, np, np] as [gate, part, out, in], np the part's width rounded
+    up to 16, zeros beyond it.  u enters the products as two bfloat16 numbers, so its first sixteen bits count."""
+    what = "rglru_gates_tc5"
+    _need_cuda(what, x, taps, conv_bias, rings, weights, gate_bias, rate, a, into, row_ids, qo_indptr, positions, state_slots, flag)
+    _need_i32(what, row_ids, qo_indptr, positions, state_slots)
+    parts = weights.shape[1]
+    T, W, n_taps = _check_rglru(what, x, taps, conv_bias, rings, gate_bias, rate, parts)
+    n = W // parts
+    np = _check_rglru_padded(what, weights, n)
+    if x.dtype != torch.bfloat16 or not rglru_tc5_supported(n):
+        raise KernelError(f"{what}: bfloat16 and parts of whole groups of eight columns")
+    for tensor in (a, into):
+        if tensor.dtype != torch.float32 or tensor.shape != (T, W) or not tensor.is_contiguous():
+            raise KernelError(f"{what}: the outputs are contiguous fp32 [tokens, width]")
+    fn = _fn("rglru_tc5", "kb_rglru_gates_tc5", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int] + [c_void_p] * 7 + [c_int] * 3 + [c_void_p, c_void_p, c_int, c_int,
+                                                                                                                                     c_void_p, c_void_p])
+    _check(fn(_tensor_map(weights.view(2 * parts * np, np), 64), x.data_ptr(), x.stride(0), taps.data_ptr(), conv_bias.data_ptr(), n_taps, _ptr(rings),
+              row_ids.data_ptr(), qo_indptr.data_ptr(), positions.data_ptr(), state_slots.data_ptr(), gate_bias.data_ptr(), rate.data_ptr(), parts, n, np,
+              a.data_ptr(), into.data_ptr(), qo_indptr.numel() - 1, T, _ptr(flag), _stream()), what)
+
+
+RGLRU_STEP_MAX_TOKENS = 128  # single-token rows up to which a step runs as one kernel (csrc/rglru.cu: rglru_step)
+
+
+def rglru_step(x: torch.Tensor, y: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, states: torch.Tensor, rings: Optional[torch.Tensor],
+               weights: torch.Tensor, gate_bias: torch.Tensor, rate: torch.Tensor, out: torch.Tensor, *, row_ids: torch.Tensor, positions: torch.Tensor,
+               state_slots: torch.Tensor, flag: Optional[torch.Tensor] = None) -> None:
+    """A step whose rows carry one token each, in one kernel (bfloat16): convolution, gates, recurrence and ``out = S gelu(y)``; ``states`` and
+    ``rings`` are left updated.  ``weights`` as ``rglru_gates_tc5`` takes them."""
+    what = "rglru_step"
+    _need_cuda(what, x, y, taps, conv_bias, states, rings, weights, gate_bias, rate, out, row_ids, positions, state_slots, flag)
+    _need_i32(what, row_ids, positions, state_slots)
+    parts = weights.shape[1]
+    T, W, n_taps = _check_rglru(what, x, taps, conv_bias, rings, gate_bias, rate, parts)
+    n = W // parts
+    np = _check_rglru_padded(what, weights, n)
+    if x.dtype != torch.bfloat16 or y.dtype != x.dtype or out.dtype != x.dtype or y.shape != x.shape or y.stride() != x.stride() or out.shape != (T, W) \
+            or not out.is_contiguous() or states.dtype != torch.float32 or states.shape[1:] != (W,) or not states.is_contiguous() or np > 4096:
+        raise KernelError(f"{what}: bfloat16 branches of one layout, a contiguous output, fp32 states [slots, width]")
+    fn = _fn("rglru", "kb_rglru_step", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int] + [c_void_p] * 8 + [c_int] * 3 + [c_void_p, c_int, c_int, c_void_p,
+                                                                                                                              c_void_p])
+    _check(fn(x.data_ptr(), y.data_ptr(), x.stride(0), taps.data_ptr(), conv_bias.data_ptr(), n_taps, states.data_ptr(), _ptr(rings), row_ids.data_ptr(),
+              positions.data_ptr(), state_slots.data_ptr(), weights.data_ptr(), gate_bias.data_ptr(), rate.data_ptr(), parts, n, np, out.data_ptr(),
+              T, T, _ptr(flag), _stream()), what)
+
+
 def rglru_scan(a: torch.Tensor, into: torch.Tensor, x: torch.Tensor, y: torch.Tensor, states: torch.Tensor, rings: Optional[torch.Tensor], n_taps: int,
                out: torch.Tensor, *, qo_indptr: torch.Tensor, positions: torch.Tensor, state_slots: torch.Tensor, segments: int = RGLRU_SEGMENTS) -> None:
     """Every row's tokens in order through S <- a S + into, ``out = S gelu(y)`` (tanh form); ``states`` [slots, width] fp32 and the rings of kept

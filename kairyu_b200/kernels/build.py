@@ -52,6 +52,7 @@ LIBRARIES: dict[str, list[str]] = {
     "delta_rule": [],
     "ssm": [],
     "rglru": [],
+    "rglru_tc5": [],
     "moe": [],
 }
 
