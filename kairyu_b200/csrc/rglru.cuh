@@ -6,17 +6,32 @@
 #define RG_MAX_TAPS 16
 
 __device__ __forceinline__ float sigmoid_exact(float z) { return 1.0f / (1.0f + expf(-z)); }
-// the same by the fast exponential and quotient (2 ulp): for the bfloat16 mode's kernels
-__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
-__device__ __forceinline__ float sqrt_fast(float x) {
+// the same by the special-function unit's exponential, reciprocal and square root (a few ulp): the bfloat16 mode's kernels
+__device__ __forceinline__ float ex2_fast(float x) {
     float y;
-    asm("sqrt.approx.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
     return y;
 }
-__device__ __forceinline__ float gelu_tanh_f(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+__device__ __forceinline__ float rcp_fast(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float sqrt_fast(float x) {
+    float y;
+    asm("sqrt.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+#define RG_LOG2E 1.4426950408889634f
+__device__ __forceinline__ float sigmoid_fast(float z) { return rcp_fast(1.0f + ex2_fast(-RG_LOG2E * z)); }
+// gelu in its tanh form, z (1 + tanh(w)) / 2 = z sigmoid(2 w)
+template <bool EXACT>
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+    const float w = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+    return EXACT ? 0.5f * z * (1.0f + tanhf(w)) : z * sigmoid_fast(2.0f * w);
+}
 
 // 1 - e^(-y) for y >= 0: the series of the exponential where the difference would cancel
-template <bool EXACT>
 __device__ __forceinline__ float one_minus_exp_neg(float y) {
     float p = -1.0f / 40320.0f;
     p = fmaf(p, y, 1.0f / 5040.0f);
@@ -26,7 +41,7 @@ __device__ __forceinline__ float one_minus_exp_neg(float y) {
     p = fmaf(p, y, 1.0f / 6.0f);
     p = fmaf(p, y, -0.5f);
     p = fmaf(p, y, 1.0f);
-    return y < 0.35f ? p * y : 1.0f - (EXACT ? expf(-y) : __expf(-y));
+    return y < 0.35f ? p * y : 1.0f - expf(-y);
 }
 
 // gate sums (biases added) and the convolved input of one channel -> the decay a and the input term
@@ -35,11 +50,18 @@ __device__ __forceinline__ void rglru_terms(float pre_r, float pre_i, float rate
     if (EXACT) {
         const float la = rate * sigmoid_exact(pre_r);
         a = expf(la);
-        into = sqrtf(one_minus_exp_neg<true>(-2.0f * la)) * sigmoid_exact(pre_i) * u;
+        into = sqrtf(one_minus_exp_neg(-2.0f * la)) * sigmoid_exact(pre_i) * u;
     } else {
         const float la = rate * sigmoid_fast(pre_r);
-        a = __expf(la);
-        into = sqrt_fast(one_minus_exp_neg<false>(-2.0f * la)) * sigmoid_fast(pre_i) * u;
+        a = ex2_fast(RG_LOG2E * la);
+        const float y = -2.0f * la;
+        // 1 - a^2, by the series while it is small (the first term left out is 2e-8 of the sum)
+        float p = fmaf(y, 1.0f / 120.0f, -1.0f / 24.0f);
+        p = fmaf(p, y, 1.0f / 6.0f);
+        p = fmaf(p, y, -0.5f);
+        p = fmaf(p, y, 1.0f);
+        const float gap = y < 0.1f ? p * y : fmaf(-a, a, 1.0f);
+        into = sqrt_fast(gap) * sigmoid_fast(pre_i) * u;
     }
 }
 

@@ -2217,23 +2217,26 @@ def ssm_gated_norm(y: torch.Tensor, x: torch.Tensor, skip: torch.Tensor, z: torc
 # ----------------------------------------------------------------------------- real-gated linear recurrent unit
 
 RGLRU_MAX_TAPS = 16
-RGLRU_SEGMENTS = 32  # warps that share a request's tokens in the walk (csrc/rglru.cu: RG_MAX_SEGMENTS)
 
 
-def _check_rglru(what: str, x: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, rings: Optional[torch.Tensor], gate_bias: torch.Tensor,
-                 rate: torch.Tensor, parts: int) -> tuple[int, int, int]:
+def _check_rglru_input(what: str, x: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, rings: Optional[torch.Tensor], parts: int) -> None:
     T, W = x.shape
     n_taps = taps.shape[0]
     if W % parts or x.stride(1) != 1:
         raise KernelError(f"{what}: {W} columns with unit inner stride in {parts} equal parts")
-    for tensor, count in ((taps, n_taps * W), (conv_bias, W), (gate_bias, 2 * W), (rate, W)):
+    for tensor, count in ((taps, n_taps * W), (conv_bias, W)):
         if tensor.dtype != torch.float32 or not tensor.is_contiguous() or tensor.numel() != count:
-            raise KernelError(f"{what}: taps [n, width], biases and rates are contiguous fp32 of the width's size")
+            raise KernelError(f"{what}: the taps [n, width] and their bias are contiguous fp32 of the width's size")
     if not 1 <= n_taps <= RGLRU_MAX_TAPS:
         raise KernelError(f"{what}: {n_taps} taps (1 to {RGLRU_MAX_TAPS})")
     if n_taps > 1 and (rings is None or rings.dtype != torch.float32 or not rings.is_contiguous() or tuple(rings.shape[1:]) != (n_taps, W)):
         raise KernelError(f"{what}: the kept inputs must be contiguous fp32 [slots, taps, width]")
-    return T, W, n_taps
+
+
+def _check_rglru_gates(what: str, gate_bias: torch.Tensor, rate: torch.Tensor, W: int) -> None:
+    for tensor, count in ((gate_bias, 2 * W), (rate, W)):
+        if tensor.dtype != torch.float32 or not tensor.is_contiguous() or tensor.numel() != count:
+            raise KernelError(f"{what}: the gates' biases [2, width] and the rates are contiguous fp32")
 
 
 def rglru_gates(x: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, rings: Optional[torch.Tensor], weights_t: torch.Tensor,
@@ -2246,7 +2249,10 @@ def rglru_gates(x: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, ri
     _need_cuda(what, x, taps, conv_bias, rings, weights_t, gate_bias, rate, a, into, row_ids, qo_indptr, positions, state_slots, flag)
     _need_i32(what, row_ids, qo_indptr, positions, state_slots)
     parts = weights_t.shape[1]
-    T, W, n_taps = _check_rglru(what, x, taps, conv_bias, rings, gate_bias, rate, parts)
+    _check_rglru_input(what, x, taps, conv_bias, rings, parts)
+    T, W = x.shape
+    n_taps = taps.shape[0]
+    _check_rglru_gates(what, gate_bias, rate, W)
     n = W // parts
     if weights_t.shape != (2, parts, n, n) or weights_t.dtype != x.dtype or not weights_t.is_contiguous():
         raise KernelError(f"{what}: the gates' matrices must be contiguous [2, parts, n, n] in x's dtype")
@@ -2260,72 +2266,97 @@ def rglru_gates(x: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, ri
               into.data_ptr(), qo_indptr.numel() - 1, T, _ptr(flag), _stream()), what)
 
 
-def rglru_tc5_supported(part_width: int) -> bool:
-    """Part widths the tensor-core kernel of the gates takes (bfloat16): whole 16-byte groups."""
-    return part_width % 8 == 0
+def rglru_padded(part_width: int) -> int:
+    """Columns a part has in what the tensor-core kernels read: its width rounded up to 16."""
+    return -(-part_width // 16) * 16
 
 
 def _check_rglru_padded(what: str, weights: torch.Tensor, n: int) -> int:
     np = weights.shape[2]
-    if weights.dtype != torch.bfloat16 or weights.dim() != 4 or weights.shape[0] != 2 or weights.shape[3] != np or np % 16 or np < n or not weights.is_contiguous():
+    if weights.dtype != torch.bfloat16 or weights.dim() != 4 or weights.shape[0] != 2 or weights.shape[3] != np or np != rglru_padded(n) or not weights.is_contiguous():
         raise KernelError(f"{what}: the gates' matrices must be contiguous bfloat16 [2, parts, np, np], np the part's width rounded up to 16")
     return np
 
 
-def rglru_gates_tc5(x: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, rings: Optional[torch.Tensor], weights: torch.Tensor,
-                    gate_bias: torch.Tensor, rate: torch.Tensor, a: torch.Tensor, into: torch.Tensor, *, row_ids: torch.Tensor, qo_indptr: torch.Tensor,
-                    positions: torch.Tensor, state_slots: torch.Tensor, flag: Optional[torch.Tensor] = None) -> None:
-    """``rglru_gates`` on tensor cores (bfloat16).  ``weights``: [2, parts, np, np] as [gate, part, out, in], np the part's width rounded
-    up to 16, zeros beyond it.  u enters the products as two bfloat16 numbers, so its first sixteen bits count."""
-    what = "rglru_gates_tc5"
-    _need_cuda(what, x, taps, conv_bias, rings, weights, gate_bias, rate, a, into, row_ids, qo_indptr, positions, state_slots, flag)
+def _check_rglru_planes(what: str, hi: torch.Tensor, lo: torch.Tensor, tokens: int, wide: int) -> None:
+    for plane in (hi, lo):
+        if plane.dtype != torch.bfloat16 or plane.shape != (tokens, wide) or not plane.is_contiguous() or plane.data_ptr() % 32:
+            raise KernelError(f"{what}: the convolved inputs are two contiguous bfloat16 planes [tokens, parts * np]")
+
+
+def rglru_convolve(x: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, rings: Optional[torch.Tensor], hi: torch.Tensor, lo: torch.Tensor, parts: int, *,
+                   row_ids: torch.Tensor, qo_indptr: torch.Tensor, positions: torch.Tensor, state_slots: torch.Tensor, update_rings: bool = False,
+                   flag: Optional[torch.Tensor] = None) -> None:
+    """The causal convolution of ``x`` [tokens, width] (bfloat16; ``taps`` [n, width] oldest first, earlier inputs from the requests' rings) as two bfloat16
+    planes [tokens, parts * np], u = hi + lo, a part's columns and then zeros up to ``rglru_padded``.  ``update_rings``: every row carries one
+    token, and its input joins its ring."""
+    what = "rglru_convolve"
+    _need_cuda(what, x, taps, conv_bias, rings, hi, lo, row_ids, qo_indptr, positions, state_slots, flag)
     _need_i32(what, row_ids, qo_indptr, positions, state_slots)
+    T, W = x.shape
+    n_taps = taps.shape[0]
+    _check_rglru_input(what, x, taps, conv_bias, rings, parts)
+    np = rglru_padded(W // parts)
+    _check_rglru_planes(what, hi, lo, T, parts * np)
+    if x.dtype != torch.bfloat16 or (update_rings and qo_indptr.numel() - 1 != T):
+        raise KernelError(f"{what}: bfloat16 inputs, and rings are updated for rows of one token only")
+    fn = _fn("rglru", "kb_rglru_convolve", [c_void_p, c_int, c_void_p, c_void_p, c_int] + [c_void_p] * 5 + [c_int] * 3 + [c_void_p, c_void_p, c_int, c_int, c_int,
+                                                                                                                      c_void_p, c_void_p])
+    _check(fn(x.data_ptr(), x.stride(0), taps.data_ptr(), conv_bias.data_ptr(), n_taps, _ptr(rings), row_ids.data_ptr(), qo_indptr.data_ptr(),
+              positions.data_ptr(), state_slots.data_ptr(), parts, W // parts, np, hi.data_ptr(), lo.data_ptr(), 1 if update_rings else 0,
+              qo_indptr.numel() - 1, T, _ptr(flag), _stream()), what)
+
+
+def rglru_gates_tc5(hi: torch.Tensor, lo: torch.Tensor, weights: torch.Tensor, gate_bias: torch.Tensor, rate: torch.Tensor, a: torch.Tensor,
+                    into: torch.Tensor, *, flag: Optional[torch.Tensor] = None) -> None:
+    """The gates of ``rglru_gates`` on tensor cores, from the planes ``rglru_convolve`` left.  ``weights``: [2, parts, np, np] as [gate, part, out, in],
+    zeros beyond a part's width."""
+    what = "rglru_gates_tc5"
+    _need_cuda(what, hi, lo, weights, gate_bias, rate, a, into, flag)
     parts = weights.shape[1]
-    T, W, n_taps = _check_rglru(what, x, taps, conv_bias, rings, gate_bias, rate, parts)
+    T, W = a.shape
     n = W // parts
     np = _check_rglru_padded(what, weights, n)
-    if x.dtype != torch.bfloat16 or not rglru_tc5_supported(n):
-        raise KernelError(f"{what}: bfloat16 and parts of whole groups of eight columns")
+    _check_rglru_planes(what, hi, lo, T, parts * np)
+    _check_rglru_gates(what, gate_bias, rate, W)
     for tensor in (a, into):
         if tensor.dtype != torch.float32 or tensor.shape != (T, W) or not tensor.is_contiguous():
             raise KernelError(f"{what}: the outputs are contiguous fp32 [tokens, width]")
-    fn = _fn("rglru_tc5", "kb_rglru_gates_tc5", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int] + [c_void_p] * 7 + [c_int] * 3 + [c_void_p, c_void_p, c_int, c_int,
-                                                                                                                                     c_void_p, c_void_p])
-    _check(fn(_tensor_map(weights.view(2 * parts * np, np), 64), x.data_ptr(), x.stride(0), taps.data_ptr(), conv_bias.data_ptr(), n_taps, _ptr(rings),
-              row_ids.data_ptr(), qo_indptr.data_ptr(), positions.data_ptr(), state_slots.data_ptr(), gate_bias.data_ptr(), rate.data_ptr(), parts, n, np,
-              a.data_ptr(), into.data_ptr(), qo_indptr.numel() - 1, T, _ptr(flag), _stream()), what)
+    fn = _fn("rglru_tc5", "kb_rglru_gates_tc5", [c_void_p] * 7 + [c_int] * 3 + [c_void_p, c_void_p, c_int, c_void_p, c_void_p])
+    _check(fn(_tensor_map(weights.view(2 * parts * np, np), 64), _tensor_map(hi, 128), _tensor_map(lo, 128), hi.data_ptr(), lo.data_ptr(),
+              gate_bias.data_ptr(), rate.data_ptr(), parts, n, np, a.data_ptr(), into.data_ptr(), T, _ptr(flag), _stream()), what)
 
 
-RGLRU_STEP_MAX_TOKENS = 128  # single-token rows up to which a step runs as one kernel (csrc/rglru.cu: rglru_step)
+RGLRU_STEP_MAX_TOKENS = 256  # single-token rows up to which gates and recurrence run as one kernel (csrc/rglru.cu: rglru_step)
 
 
-def rglru_step(x: torch.Tensor, y: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor, states: torch.Tensor, rings: Optional[torch.Tensor],
-               weights: torch.Tensor, gate_bias: torch.Tensor, rate: torch.Tensor, out: torch.Tensor, *, row_ids: torch.Tensor, positions: torch.Tensor,
-               state_slots: torch.Tensor, flag: Optional[torch.Tensor] = None) -> None:
-    """A step whose rows carry one token each, in one kernel (bfloat16): convolution, gates, recurrence and ``out = S gelu(y)``; ``states`` and
-    ``rings`` are left updated.  ``weights`` as ``rglru_gates_tc5`` takes them."""
+def rglru_step(hi: torch.Tensor, lo: torch.Tensor, y: torch.Tensor, states: torch.Tensor, weights: torch.Tensor, gate_bias: torch.Tensor, rate: torch.Tensor,
+               out: torch.Tensor, *, row_ids: torch.Tensor, state_slots: torch.Tensor, flag: Optional[torch.Tensor] = None) -> None:
+    """Gates and recurrence of a step whose rows carry one token each, from the planes ``rglru_convolve`` left (which has updated the rings):
+    ``out = S gelu(y)``, ``states`` left updated.  ``weights`` as ``rglru_gates_tc5`` takes them."""
     what = "rglru_step"
-    _need_cuda(what, x, y, taps, conv_bias, states, rings, weights, gate_bias, rate, out, row_ids, positions, state_slots, flag)
-    _need_i32(what, row_ids, positions, state_slots)
+    _need_cuda(what, hi, lo, y, states, weights, gate_bias, rate, out, row_ids, state_slots, flag)
+    _need_i32(what, row_ids, state_slots)
     parts = weights.shape[1]
-    T, W, n_taps = _check_rglru(what, x, taps, conv_bias, rings, gate_bias, rate, parts)
+    T, W = out.shape
     n = W // parts
     np = _check_rglru_padded(what, weights, n)
-    if x.dtype != torch.bfloat16 or y.dtype != x.dtype or out.dtype != x.dtype or y.shape != x.shape or y.stride() != x.stride() or out.shape != (T, W) \
-            or not out.is_contiguous() or states.dtype != torch.float32 or states.shape[1:] != (W,) or not states.is_contiguous() or np > 4096:
-        raise KernelError(f"{what}: bfloat16 branches of one layout, a contiguous output, fp32 states [slots, width]")
-    fn = _fn("rglru", "kb_rglru_step", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int] + [c_void_p] * 8 + [c_int] * 3 + [c_void_p, c_int, c_int, c_void_p,
-                                                                                                                              c_void_p])
-    _check(fn(x.data_ptr(), y.data_ptr(), x.stride(0), taps.data_ptr(), conv_bias.data_ptr(), n_taps, states.data_ptr(), _ptr(rings), row_ids.data_ptr(),
-              positions.data_ptr(), state_slots.data_ptr(), weights.data_ptr(), gate_bias.data_ptr(), rate.data_ptr(), parts, n, np, out.data_ptr(),
-              T, T, _ptr(flag), _stream()), what)
+    _check_rglru_planes(what, hi, lo, T, parts * np)
+    _check_rglru_gates(what, gate_bias, rate, W)
+    if y.dtype != torch.bfloat16 or out.dtype != y.dtype or y.shape != out.shape or y.stride(1) != 1 or not out.is_contiguous() or states.dtype != torch.float32 \
+            or states.shape[1:] != (W,) or not states.is_contiguous() or row_ids.numel() != T:
+        raise KernelError(f"{what}: a bfloat16 branch, a contiguous output, fp32 states [slots, width], a row a token")
+    fn = _fn("rglru", "kb_rglru_step", [c_void_p, c_void_p, c_void_p, c_int] + [c_void_p] * 6 + [c_int] * 3 + [c_void_p, c_int, c_int, c_void_p, c_void_p])
+    _check(fn(hi.data_ptr(), lo.data_ptr(), y.data_ptr(), y.stride(0), states.data_ptr(), row_ids.data_ptr(), state_slots.data_ptr(), weights.data_ptr(),
+              gate_bias.data_ptr(), rate.data_ptr(), parts, n, np, out.data_ptr(), T, T, _ptr(flag), _stream()), what)
 
 
 def rglru_scan(a: torch.Tensor, into: torch.Tensor, x: torch.Tensor, y: torch.Tensor, states: torch.Tensor, rings: Optional[torch.Tensor], n_taps: int,
-               out: torch.Tensor, *, qo_indptr: torch.Tensor, positions: torch.Tensor, state_slots: torch.Tensor, segments: int = RGLRU_SEGMENTS) -> None:
+               out: torch.Tensor, *, qo_indptr: torch.Tensor, positions: torch.Tensor, state_slots: torch.Tensor, segments: Optional[tuple[int, int]] = None) -> None:
     """Every row's tokens in order through S <- a S + into, ``out = S gelu(y)`` (tanh form); ``states`` [slots, width] fp32 and the rings of kept
-    inputs [slots, taps, width] are left updated.  ``x`` and ``y``: the two branches' columns of the packed projection.  ``segments``: warps
-    that share a row's tokens (1: the plain walk, whose rounding does not depend on how a prompt was cut)."""
+    inputs [slots, taps, width] are left updated.  ``x`` and ``y``: the two branches' columns of the packed projection.  ``segments``: (warps of a
+    block, blocks of a cluster) that share a row's tokens; (1, 1): the plain walk, whose rounding does not depend on how a prompt was cut; None:
+    chosen from the width and the number of tokens."""
     what = "rglru_scan"
     _need_cuda(what, a, into, x, y, states, rings, out, qo_indptr, positions, state_slots)
     _need_i32(what, qo_indptr, positions, state_slots)
@@ -2336,9 +2367,10 @@ def rglru_scan(a: torch.Tensor, into: torch.Tensor, x: torch.Tensor, y: torch.Te
     if into.shape != a.shape or x.shape != a.shape or y.shape != a.shape or x.stride() != y.stride() or x.stride(1) != 1 or x.dtype != y.dtype or out.dtype != x.dtype \
             or out.shape != a.shape or not out.is_contiguous() or states.shape[1:] != (W,) or (n_taps > 1 and (rings is None or tuple(rings.shape[1:]) != (n_taps, W))):
         raise KernelError(f"{what}: shape or dtype mismatch")
-    fn = _fn("rglru", "kb_rglru_scan", [c_void_p] * 4 + [c_int] * 4 + [c_void_p] * 6 + [c_int, c_int, c_void_p])
+    warps, cluster = segments if segments is not None else (0, 0)
+    fn = _fn("rglru", "kb_rglru_scan", [c_void_p] * 4 + [c_int] * 4 + [c_void_p] * 6 + [c_int, c_int, c_int, c_int, c_void_p])
     _check(fn(a.data_ptr(), into.data_ptr(), x.data_ptr(), y.data_ptr(), x.stride(0), _is_bf16(x, what), W, int(n_taps), states.data_ptr(), _ptr(rings),
-              qo_indptr.data_ptr(), positions.data_ptr(), state_slots.data_ptr(), out.data_ptr(), qo_indptr.numel() - 1, int(segments), _stream()), what)
+              qo_indptr.data_ptr(), positions.data_ptr(), state_slots.data_ptr(), out.data_ptr(), qo_indptr.numel() - 1, T, int(warps), int(cluster), _stream()), what)
 
 
 # ----------------------------------------------------------------------------- mixture of experts

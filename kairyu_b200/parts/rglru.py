@@ -58,8 +58,8 @@ class RealGatedLRU(Mixer):
         self.b_in: Optional[torch.Tensor] = None
         self.taps: Optional[torch.Tensor] = None        # [taps, width]
         self.conv_bias: Optional[torch.Tensor] = None
-        self.gates: Optional[torch.Tensor] = None       # tensor-core kernels: [2, parts, np, np] as [gate, part, out, in], n rounded up to 16
-        self.gates_t: Optional[torch.Tensor] = None     # else: [2, parts, n, n] as [gate, part, in, out]
+        self.gates: Optional[torch.Tensor] = None       # bfloat16: [2, parts, np, np] as [gate, part, out, in], n rounded up to 16
+        self.gates_t: Optional[torch.Tensor] = None     # float32: [2, parts, n, n] as [gate, part, in, out]
         self.gate_bias: Optional[torch.Tensor] = None   # [2, width]
         self.rate: Optional[torch.Tensor] = None        # [width]: -8 softplus(lam)
         self.w_o: Optional[torch.Tensor] = None
@@ -84,10 +84,10 @@ class RealGatedLRU(Mixer):
         gates = torch.stack([tensors[f"{p}.ra"], tensors[f"{p}.ri"]])
         n = self.width // self.parts
         if self.dtype == torch.bfloat16:
-            padded = -(-n // 16) * 16
+            padded = kernels.rglru_padded(n)
             self.gates = torch.zeros((2, self.parts, padded, padded), dtype=gates.dtype, device=gates.device)
             self.gates[:, :, :n, :n] = gates
-        if not self._tensor_cores():
+        else:
             self.gates_t = gates.transpose(2, 3).contiguous()
         self.gate_bias = torch.stack([tensors[f"{p}.ra.b"].float().reshape(-1), tensors[f"{p}.ri.b"].float().reshape(-1)]).contiguous()
         lam = tensors[f"{p}.lam"].double()
@@ -98,10 +98,6 @@ class RealGatedLRU(Mixer):
         gates = self.gates if self.gates is not None else self.gates_t
         held = (self.w_in, self.b_in, self.taps, self.conv_bias, gates, self.gate_bias, self.rate, self.w_o)
         return sum(t.numel() * t.element_size() for t in held)
-
-    def _tensor_cores(self) -> bool:
-        """Whether the gates of a step with prompt portions run on tensor cores."""
-        return self.dtype == torch.bfloat16 and kernels.rglru_tc5_supported(self.width // self.parts)
 
     def cache_specs(self) -> tuple[Any, ...]:
         specs = [StateSpec((self.width,), "float32")]
@@ -125,20 +121,25 @@ class RealGatedLRU(Mixer):
         kernels.linear(x, self.w_in, self.b_in, packed)
         y_branch, x_branch = packed[:, : self.width], packed[:, self.width :]
         mixed = ws.buffer("rglru.mixed", tokens, self.width, self.dtype)
-        step = dict(row_ids=ctx.row_ids, positions=ctx.positions, state_slots=ctx.state_slots)
-        single = tokens == ctx.num_rows  # every row carries one token
-        if single and self.gates is not None and tokens <= kernels.RGLRU_STEP_MAX_TOKENS:
-            kernels.rglru_step(x_branch, y_branch, self.taps, self.conv_bias, memory, rings, self.gates, self.gate_bias, self.rate, mixed,
-                               flag=ctx.error_flag, **step)
-        else:
+        slots = dict(row_ids=ctx.row_ids, state_slots=ctx.state_slots)
+        step = dict(slots, qo_indptr=ctx.qo_indptr, positions=ctx.positions)
+        single = tokens == ctx.num_rows and tokens <= kernels.RGLRU_STEP_MAX_TOKENS  # every row carries one token
+        if self.gates is not None:
+            wide = self.parts * self.gates.shape[2]
+            hi, lo = (ws.buffer(f"rglru.{name}", tokens, wide, self.dtype) for name in ("hi", "lo"))
+            kernels.rglru_convolve(x_branch, self.taps, self.conv_bias, rings, hi, lo, self.parts, update_rings=single, flag=ctx.error_flag, **step)
+            if single:
+                kernels.rglru_step(hi, lo, y_branch, memory, self.gates, self.gate_bias, self.rate, mixed, flag=ctx.error_flag, **slots)
+        if self.gates is None or not single:
             a = ws.buffer("rglru.a", tokens, self.width, torch.float32)
             into = ws.buffer("rglru.into", tokens, self.width, torch.float32)
-            gates, weights = (kernels.rglru_gates_tc5, self.gates) if self._tensor_cores() else (kernels.rglru_gates, self.gates_t)
-            gates(x_branch, self.taps, self.conv_bias, rings, weights, self.gate_bias, self.rate, a, into, qo_indptr=ctx.qo_indptr, flag=ctx.error_flag, **step)
+            if self.gates is not None:
+                kernels.rglru_gates_tc5(hi, lo, self.gates, self.gate_bias, self.rate, a, into, flag=ctx.error_flag)
+            else:
+                kernels.rglru_gates(x_branch, self.taps, self.conv_bias, rings, self.gates_t, self.gate_bias, self.rate, a, into, flag=ctx.error_flag, **step)
             # 32-bit mode walks a request's tokens one by one, so that a result does not depend on where a prompt was cut
-            segments = 1 if self.dtype == torch.float32 or single else kernels.RGLRU_SEGMENTS
             kernels.rglru_scan(a, into, x_branch, y_branch, memory, rings, self.conv_taps, mixed, qo_indptr=ctx.qo_indptr, positions=ctx.positions,
-                               state_slots=ctx.state_slots, segments=segments)
+                               state_slots=ctx.state_slots, segments=(1, 1) if self.dtype == torch.float32 else None)
         if fold is not None:
             kernels.linear(mixed, self.w_o, None, None, fold=fold)
             return fold.result()
