@@ -395,9 +395,12 @@ projection_norm_rope_write_vec_kernel(__nv_bfloat16* __restrict__ packed, int st
     }
 }
 
-// The same with statistics a head, or none, on bfloat16 rows of whole 16-byte groups: GROUP lanes hold a head in registers
-// (eight columns a lane), so a head is read once, its sum is a butterfly among its lanes and nothing waits for another head.
-// A value head is an item of its own, or (values that are the keys as projected) goes out with its key.
+// The same with statistics a head, or none, on bfloat16 rows of whole 16-byte groups: GROUP lanes hold PR_GROUP_HEADS heads of a token in
+// registers (eight columns a lane and head), so a head is read once, its sum is a butterfly among its lanes, the token's angles
+// are fetched once for all of them and nothing waits for another head.  A value head is one of the heads, or (values that are
+// the keys as projected) goes out with its key.
+#define PR_GROUP_HEADS 4
+
 template <int GROUP, typename TW>
 __global__ void __launch_bounds__(PR_THREADS)
 head_norm_rope_write_kernel(__nv_bfloat16* __restrict__ packed, int stride, int k_offset, int v_offset, int Hq, int Hkv, int D, int DV,
@@ -406,22 +409,21 @@ head_norm_rope_write_kernel(__nv_bfloat16* __restrict__ packed, int stride, int 
                             int interleaved, const int* __restrict__ positions, const int* __restrict__ row_ids,
                             const int* __restrict__ block_table, int max_pages, const int* __restrict__ write_from,
                             __nv_bfloat16* __restrict__ k_cache, __nv_bfloat16* __restrict__ v_cache, int page_size, int num_pages,
-                            int num_rows, int T, int* flag) {
+                            int num_rows, int T, int heads, int* flag) {
     pdl_trigger();
     const bool keys_are_values = v_offset == k_offset && DV == D;
-    const int heads = Hq + Hkv + (k_cache && !keys_are_values ? Hkv : 0);
+    const int bundles = (heads + PR_GROUP_HEADS - 1) / PR_GROUP_HEADS;
     const long long item = ((long long)blockIdx.x * PR_THREADS + threadIdx.x) / GROUP;
-    const int j = threadIdx.x % GROUP;  // this lane's eight columns of the head
-    const bool live = item < (long long)T * heads;
-    const int t = live ? (int)(item / heads) : 0;
-    const int head = live ? (int)(item % heads) : 0;
-    const bool is_q = head < Hq, is_v = head >= Hq + Hkv;
+    const int j = threadIdx.x % GROUP;  // this lane's eight columns of each head
+    const bool live = item < (long long)T * bundles;
+    const int t = live ? (int)(item / bundles) : 0;
+    const int head0 = live ? (int)(item % bundles) * PR_GROUP_HEADS : heads;
     const int pos = positions[t];
     const bool pos_ok = rot_half == 0 || (pos >= 0 && pos < max_pos);
-    // where a key or value row goes (negative: nowhere)
+    // where the token's key and value rows go (negative: nowhere)
     long long place = -1;
     int trouble = pos_ok ? 0 : KB_FLAG_BAD_POS;
-    if (!is_q && k_cache) {
+    if (k_cache && head0 + PR_GROUP_HEADS > Hq && live) {
         const int row = row_ids[t];
         if (row < 0 || row >= num_rows) {
             trouble |= KB_FLAG_BAD_ROW;
@@ -432,11 +434,9 @@ head_norm_rope_write_kernel(__nv_bfloat16* __restrict__ packed, int stride, int 
             else place = (long long)page * page_size + (pos % page_size);
         }
     }
-    const int groups = (is_v ? DV : D) / 8;
-    const bool holds = live && j < groups;
     // this lane's angles: of pair (i, i + rot_half) for both of the lanes that hold its two sides; of four pairs when interleaved
     const int rot_groups = interleaved ? rot_half / 4 : rot_half / 8;
-    const bool turns = holds && !is_v && j < (interleaved ? rot_groups : 2 * rot_groups);
+    const bool turns = live && j < (interleaved ? rot_groups : 2 * rot_groups);
     float c8[8], s8[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
@@ -454,76 +454,89 @@ head_norm_rope_write_kernel(__nv_bfloat16* __restrict__ packed, int stride, int 
             load_floats(sn + (j % rot_groups) * 8, 8, s8);
         }
     }
+    // the lane that holds the other side of its pairs (split halves); lanes that turn nothing exchange with themselves
+    const bool first = j < rot_groups;
+    const int partner = (threadIdx.x & 31) + (turns && !interleaved ? (first ? rot_groups : -rot_groups) : 0);
     pdl_wait();
     if (live && j == 0 && trouble && flag) atomicOr(flag, trouble);
-    const int local = is_q ? head : (is_v ? head - Hq - Hkv : head - Hq);
-    __nv_bfloat16* src = packed + (size_t)t * stride + (is_q ? 0 : is_v ? v_offset : k_offset) + local * (is_v ? DV : D) + j * 8;
-    Bf16x8 raw;
-#pragma unroll
-    for (int e = 0; e < 4; ++e) raw.v[e] = __floats2bfloat162_rn(0.0f, 0.0f);
-    if (holds) raw = *reinterpret_cast<const Bf16x8*>(src);
-    float a[8];
-    unpack8(raw, a);
-    auto sum_of_squares = [&]() -> float {
-        float ss = 0.0f;
-#pragma unroll
-        for (int e = 0; e < 8; ++e) ss += a[e] * a[e];
-#pragma unroll
-        for (int offset = GROUP / 2; offset > 0; offset >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, offset);
-        return ss;
+    __nv_bfloat16* row_of = packed + (size_t)t * stride + j * 8;
+    auto source = [&](int head) -> __nv_bfloat16* {
+        if (head < Hq) return row_of + head * D;
+        if (head < Hq + Hkv) return row_of + k_offset + (head - Hq) * D;
+        return row_of + v_offset + (head - Hq - Hkv) * DV;
     };
-    if (wq) {
-        const float inv = rsqrtf(sum_of_squares() / (float)D + eps);
-        if (holds && !is_v) {
-            float w8[8];
-            load_weights8(is_q ? wq : wk, j * 8, inv, w8);
+    Bf16x8 raw[PR_GROUP_HEADS];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) a[e] *= w8[e];
-        }
+    for (int i = 0; i < PR_GROUP_HEADS; ++i) {
+        const int head = head0 + i;
+        const bool holds = head < heads && j < (head < Hq + Hkv ? D : DV) / 8;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) raw[i].v[e] = __floats2bfloat162_rn(0.0f, 0.0f);
+        if (holds) raw[i] = *reinterpret_cast<const Bf16x8*>(source(head));
     }
-    if (interleaved) {
-        if (turns) {
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                float rx, ry;
-                rotate(a[2 * e], a[2 * e + 1], c8[e], s8[e], rx, ry);
-                a[2 * e] = rx;
-                a[2 * e + 1] = ry;
+    for (int i = 0; i < PR_GROUP_HEADS; ++i) {
+        const int head = head0 + i;
+        const bool is_q = head < Hq, is_v = head >= Hq + Hkv;
+        const bool holds = head < heads && j < (is_v ? DV : D) / 8;
+        float a[8];
+        unpack8(raw[i], a);
+        auto sum_of_squares = [&]() -> float {
+            float ss = 0.0f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss += a[e] * a[e];
+#pragma unroll
+            for (int offset = GROUP / 2; offset > 0; offset >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, offset);
+            return ss;
+        };
+        if (wq) {
+            const float inv = rsqrtf(sum_of_squares() / (float)D + eps);
+            if (holds && !is_v) {
+                float w8[8];
+                load_weights8(is_q ? wq : wk, j * 8, inv, w8);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) a[e] *= w8[e];
             }
         }
-    } else if (rot_half > 0) {
-        // the lane that holds the other side of these pairs; lanes that turn nothing exchange with themselves
-        const bool first = j < rot_groups;
-        const int lane = threadIdx.x & 31;
-        const int partner = turns ? lane + (first ? rot_groups : -rot_groups) : lane;
+        if (interleaved) {
+            if (turns) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-            const float other = __shfl_sync(0xffffffffu, a[e], partner);
-            float rx, ry;
-            rotate(first ? a[e] : other, first ? other : a[e], c8[e], s8[e], rx, ry);
-            if (turns) a[e] = first ? rx : ry;
+                for (int e = 0; e < 4; ++e) {
+                    float rx, ry;
+                    rotate(a[2 * e], a[2 * e + 1], c8[e], s8[e], rx, ry);
+                    a[2 * e] = rx;
+                    a[2 * e + 1] = ry;
+                }
+            }
+        } else if (rot_half > 0) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                const float other = __shfl_sync(0xffffffffu, a[e], partner);
+                float rx, ry;
+                rotate(first ? a[e] : other, first ? other : a[e], c8[e], s8[e], rx, ry);
+                if (turns) a[e] = first ? rx : ry;
+            }
         }
-    }
-    if (norm_after) {
-        const float inv = rsqrtf(sum_of_squares() / (float)D + eps);
-        if (!is_v) {
+        if (norm_after) {
+            const float inv = rsqrtf(sum_of_squares() / (float)D + eps);
 #pragma unroll
             for (int e = 0; e < 8; ++e) a[e] *= inv;
         }
-    }
-    if (!holds) return;
-    if (turns && !pos_ok) {
+        if (!holds) continue;
+        if (turns && !pos_ok) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) a[e] = 0.0f;
-    }
-    if (is_q) {
-        *reinterpret_cast<Bf16x8*>(src) = pack8(a);
-    } else if (place >= 0) {
-        if (is_v) {
-            *reinterpret_cast<Bf16x8*>(v_cache + ((size_t)place * Hkv + local) * DV + j * 8) = raw;
-        } else {
-            *reinterpret_cast<Bf16x8*>(k_cache + ((size_t)place * Hkv + local) * D + j * 8) = pack8(a);
-            if (keys_are_values) *reinterpret_cast<Bf16x8*>(v_cache + ((size_t)place * Hkv + local) * D + j * 8) = raw;
+            for (int e = 0; e < 8; ++e) a[e] = 0.0f;
+        }
+        if (is_q) {
+            *reinterpret_cast<Bf16x8*>(source(head)) = pack8(a);
+        } else if (place >= 0) {
+            const int local = is_v ? head - Hq - Hkv : head - Hq;
+            if (is_v) {
+                *reinterpret_cast<Bf16x8*>(v_cache + ((size_t)place * Hkv + local) * DV + j * 8) = raw[i];
+            } else {
+                *reinterpret_cast<Bf16x8*>(k_cache + ((size_t)place * Hkv + local) * D + j * 8) = pack8(a);
+                if (keys_are_values) *reinterpret_cast<Bf16x8*>(v_cache + ((size_t)place * Hkv + local) * D + j * 8) = raw[i];
+            }
         }
     }
 }
@@ -565,14 +578,16 @@ KB_EXPORT int kb_projection_norm_rope_write(void* packed, int stride, int is_bf1
     kb_launch(head_norm_rope_write_kernel<GROUP, TW>, dim3((unsigned)((items * GROUP + PR_THREADS - 1) / PR_THREADS)), dim3(PR_THREADS), 0,  \
               stream, (__nv_bfloat16*)packed, stride, k_offset, v_offset, Hq, Hkv, D, DV, (const TW*)wq, (const TW*)wk, eps, norm_after,  \
               cos_table, sin_table, rot_half, max_pos, interleaved, positions, row_ids, block_table, max_pages, write_from,         \
-              (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, page_size, num_pages, num_rows, T, flag)
+              (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, page_size, num_pages, num_rows, T, heads, flag)
 #define PICK_HEADS(TW)                                                                                                              \
     do {                                                                                                                            \
         if (lanes <= 4) LAUNCH_HEADS(4, TW); else if (lanes <= 8) LAUNCH_HEADS(8, TW);                                              \
         else if (lanes <= 16) LAUNCH_HEADS(16, TW); else LAUNCH_HEADS(32, TW);                                                      \
     } while (0)
     const int lanes = (k_cache && DV > D ? DV : D) / 8;  // 16-byte groups of the widest head
-    const long long items = (long long)T * (Hq + Hkv + (k_cache && !(v_offset == k_offset && DV == D) ? Hkv : 0));
+    // heads of a token: a value head counts where it is not its key
+    const int heads = Hq + Hkv + (k_cache && !(v_offset == k_offset && DV == D) ? Hkv : 0);
+    const long long items = (long long)T * ((heads + PR_GROUP_HEADS - 1) / PR_GROUP_HEADS);
     if (groups_of_eight && (per_head || !wq) && v_rot_half == 0 && lanes <= 32 && items < (1ll << 27)) {
         if (w_bf16) PICK_HEADS(__nv_bfloat16); else PICK_HEADS(float);
     } else if (groups_of_eight && !norm_after) {

@@ -112,7 +112,7 @@ def latent_attention(h, w, m, eps):
 def short_convolution(x, taps, bias):
     """y_t = b + sum_j taps[:, last - j] * x_(t - j), zeros before the start."""
     y = bias.expand_as(x).clone()
-    for back in range(taps.shape[1]):
+    for back in range(min(taps.shape[1], x.shape[0])):
         y[back:] += taps[:, taps.shape[1] - 1 - back] * x[: x.shape[0] - back]
     return y
 
