@@ -63,22 +63,7 @@ __global__ void embedding_norm_kernel(const TT* __restrict__ table, const int* _
     }
 }
 
-KB_EXPORT int kb_embedding_norm(const void* table, int table_is_bf16, const int* ids, const void* w, int w_is_bf16, float* out, float* origin,
-                                int T, int H, int V, float scale, float eps, int* flag, cudaStream_t stream) {
-    if (T == 0) return 0;
-    if (!table || !ids || !out) return KB_ERR_NULL;
-    const int threads = H >= 1024 ? 256 : 128;
-#define LAUNCH(TT, TW)                                                                                                                   \
-    kb_launch(embedding_norm_kernel<TT, TW>, dim3(T), dim3(threads), 0, stream, (const TT*)table, ids, (const TW*)w, out, origin, H, V, scale, \
-              eps, flag)
-    if (table_is_bf16) {
-        if (w_is_bf16) LAUNCH(__nv_bfloat16, __nv_bfloat16); else LAUNCH(__nv_bfloat16, float);
-    } else {
-        if (w_is_bf16) LAUNCH(float, __nv_bfloat16); else LAUNCH(float, float);
-    }
-#undef LAUNCH
-    return kb_launch_result();
-}
+// (the entry point follows the vector helpers further down)
 
 // ------------------------------------------------------------------ learned positions
 // x[t, :] += table[positions[t], :] on the fp32 residual.  A position outside [0, P) adds nothing
@@ -217,6 +202,70 @@ struct Vec4<__nv_bfloat16> {
         *reinterpret_cast<uint2*>(p) = r;
     }
 };
+
+// ---- the embedding with a norm of its own: rows of whole groups of four, held in registers between the sum and the store, every load in
+// flight at once (the scalar kernel above reads a row twice)
+template <typename TT, typename TW>
+__global__ void __launch_bounds__(1024)
+embedding_norm_vec_kernel(const TT* __restrict__ table, const int* __restrict__ ids, const TW* __restrict__ w, float* __restrict__ out,
+                          float* __restrict__ origin, int H, int V, float scale, float eps, int* flag) {
+    __shared__ float scratch[32];
+    const int t = blockIdx.x;
+    pdl_wait();
+    const int id = ids[t];
+    const bool known = id >= 0 && id < V;
+    if (!known && threadIdx.x == 0 && flag) atomicOr(flag, KB_FLAG_BAD_TOKEN);
+    const TT* src = table + (size_t)(known ? id : 0) * H;
+    float v[NORM_MAX_CHUNKS][4], wv[NORM_MAX_CHUNKS][4];
+    float ss = 0.0f;
+#pragma unroll
+    for (int c = 0; c < NORM_MAX_CHUNKS; ++c) {
+        const int at = (threadIdx.x + c * blockDim.x) * 4;
+        if (at < H) {
+            Vec4<TT>::load(src + at, v[c]);
+            if (w) Vec4<TW>::load(w + at, wv[c]);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                v[c][e] = known ? v[c][e] * scale : 0.0f;
+                ss += v[c][e] * v[c][e];
+            }
+        }
+    }
+    const float inv = w ? rsqrtf(block_sum(ss, scratch) / (float)H + eps) : 1.0f;
+#pragma unroll
+    for (int c = 0; c < NORM_MAX_CHUNKS; ++c) {
+        const int at = (threadIdx.x + c * blockDim.x) * 4;
+        if (at < H) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[c][e] *= w ? inv * wv[c][e] : 1.0f;
+            Vec4<float>::store(out + (size_t)t * H + at, v[c]);
+            if (origin) Vec4<float>::store(origin + (size_t)t * H + at, v[c]);
+        }
+    }
+}
+
+KB_EXPORT int kb_embedding_norm(const void* table, int table_is_bf16, const int* ids, const void* w, int w_is_bf16, float* out, float* origin,
+                                int T, int H, int V, float scale, float eps, int* flag, cudaStream_t stream) {
+    if (T == 0) return 0;
+    if (!table || !ids || !out) return KB_ERR_NULL;
+    const bool vec = H % 4 == 0 && H <= 16 * 1024 && ((uintptr_t)table | (uintptr_t)w | (uintptr_t)out | (uintptr_t)origin) % 16 == 0;
+    int threads = H >= 1024 ? 256 : 128;
+    if (vec) threads = H > 4096 ? 1024 : (H / 4 + 31) / 32 * 32;
+#define LAUNCH(KERNEL, TT, TW)                                                                                                           \
+    kb_launch(KERNEL<TT, TW>, dim3(T), dim3(threads), 0, stream, (const TT*)table, ids, (const TW*)w, out, origin, H, V, scale, eps, flag)
+#define PICK(KERNEL)                                                                                                                      \
+    do {                                                                                                                                  \
+        if (table_is_bf16) {                                                                                                              \
+            if (w_is_bf16) LAUNCH(KERNEL, __nv_bfloat16, __nv_bfloat16); else LAUNCH(KERNEL, __nv_bfloat16, float);                        \
+        } else {                                                                                                                          \
+            if (w_is_bf16) LAUNCH(KERNEL, float, __nv_bfloat16); else LAUNCH(KERNEL, float, float);                                        \
+        }                                                                                                                                 \
+    } while (0)
+    if (vec) PICK(embedding_norm_vec_kernel); else PICK(embedding_norm_kernel);
+#undef PICK
+#undef LAUNCH
+    return kb_launch_result();
+}
 
 // ---- the activation kernels (unary_activation is defined with the feed-forward's activations above)
 template <typename T>

@@ -201,7 +201,7 @@ rglru_scan_kernel(const float* __restrict__ a_in, const float* __restrict__ into
 // hi, lo: [tokens, parts * np], a part's n columns and zeros behind them (np: n rounded up to 16): u = hi + lo to sixteen bits and more.
 // VEC: a thread takes eight channels of RG_CONV_TOKENS consecutive tokens; else one channel of one token.  `single`: every row
 // carries one token; the kernel then also writes the token's input to its ring (a row none of its reads touches).
-#define RG_CONV_TOKENS 4
+#define RG_CONV_TOKENS 2
 
 __device__ __forceinline__ void rg_split(float u, __nv_bfloat16& hi, __nv_bfloat16& lo) {
     hi = __float2bfloat16_rn(u);
@@ -494,12 +494,13 @@ KB_EXPORT int kb_rglru_scan(const float* a, const float* into, const void* x, co
     if (W < 1 || n_taps < 1 || n_taps > RG_MAX_TAPS || num_rows > 65535) return KB_ERR_BAD_ARG;
     if (n_taps > 1 && !rings) return KB_ERR_NULL;
     if (warps == 0 && cluster == 0) {
-        // segments of sixteen tokens and more of an average row, and no more blocks than two a SM
+        // segments of sixteen tokens and more of an average row; blocks until there are two for most SMs (2,048 tokens: width 2,048 takes 27 us with
+        // clusters of four, 33 of eight, 53 of one; width 4,096 45 with clusters of two, 49 of four, 61 of one)
         const int groups = (W + 31) / 32;
         long long segments = ((long long)T / num_rows + 15) / 16;
         warps = segments < 1 ? 1 : segments > RG_MAX_WARPS ? RG_MAX_WARPS : (int)segments;
         cluster = 1;
-        while (cluster < RG_MAX_CLUSTER && segments >= 2 * cluster * warps && (long long)groups * num_rows * cluster * 2 <= 4 * 148) cluster *= 2;
+        while (cluster < RG_MAX_CLUSTER && segments >= 2 * cluster * warps && (long long)groups * num_rows * cluster * 2 <= 2 * 148) cluster *= 2;
     }
     if (warps < 1 || warps > RG_MAX_WARPS || cluster < 1 || cluster > RG_MAX_CLUSTER || (cluster & (cluster - 1)) != 0) return KB_ERR_BAD_ARG;
     cudaLaunchConfig_t config = {};

@@ -31,37 +31,28 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
     return EXACT ? 0.5f * z * (1.0f + tanhf(w)) : z * sigmoid_fast(2.0f * w);
 }
 
-// 1 - e^(-y) for y >= 0: the series of the exponential where the difference would cancel
-__device__ __forceinline__ float one_minus_exp_neg(float y) {
-    float p = -1.0f / 40320.0f;
-    p = fmaf(p, y, 1.0f / 5040.0f);
-    p = fmaf(p, y, -1.0f / 720.0f);
-    p = fmaf(p, y, 1.0f / 120.0f);
-    p = fmaf(p, y, -1.0f / 24.0f);
-    p = fmaf(p, y, 1.0f / 6.0f);
-    p = fmaf(p, y, -0.5f);
-    p = fmaf(p, y, 1.0f);
-    return y < 0.35f ? p * y : 1.0f - expf(-y);
-}
-
-// gate sums (biases added) and the convolved input of one channel -> the decay a and the input term
+// Gate sums (biases added) and the convolved input of one channel -> the decay a and the input term.  What matters of a decay close to
+// one is its distance d = 1 - a from one: a rounding of a that leans one way is one of d multiplied by 1 / d, and every token of a long
+// memory adds it again.  So d comes first, without the cancellation, a is 1 - d rounded once, and 1 - a^2 = d (2 - d).
 template <bool EXACT>
 __device__ __forceinline__ void rglru_terms(float pre_r, float pre_i, float rate, float u, float& a, float& into) {
     if (EXACT) {
         const float la = rate * sigmoid_exact(pre_r);
-        a = expf(la);
-        into = sqrtf(one_minus_exp_neg(-2.0f * la)) * sigmoid_exact(pre_i) * u;
+        const float d = -expm1f(la);
+        a = la > -0.5f ? 1.0f - d : expf(la);
+        into = sqrtf(d * (2.0f - d)) * sigmoid_exact(pre_i) * u;
     } else {
-        const float la = rate * sigmoid_fast(pre_r);
-        a = ex2_fast(RG_LOG2E * la);
-        const float y = -2.0f * la;
-        // 1 - a^2, by the series while it is small (the first term left out is 2e-8 of the sum)
-        float p = fmaf(y, 1.0f / 120.0f, -1.0f / 24.0f);
-        p = fmaf(p, y, 1.0f / 6.0f);
-        p = fmaf(p, y, -0.5f);
-        p = fmaf(p, y, 1.0f);
-        const float gap = y < 0.1f ? p * y : fmaf(-a, a, 1.0f);
-        into = sqrt_fast(gap) * sigmoid_fast(pre_i) * u;
+        const float x = -rate * sigmoid_fast(pre_r);
+        // 1 - e^(-x), by its series while it is small (the first term left out is 2e-8 of the sum)
+        float p = fmaf(x, 1.0f / 120.0f, -1.0f / 24.0f);
+        p = fmaf(p, x, 1.0f / 6.0f);
+        p = fmaf(p, x, -0.5f);
+        p = fmaf(p, x, 1.0f);
+        const float far = ex2_fast(-RG_LOG2E * x);
+        const bool small = x < 0.1f;
+        const float d = small ? p * x : 1.0f - far;
+        a = small ? 1.0f - d : far;
+        into = sqrt_fast(d * (2.0f - d)) * sigmoid_fast(pre_i) * u;
     }
 }
 

@@ -277,7 +277,7 @@ def test_plain_model_pieces():
     for i in range(8):
         share = min(max((i - lo) / (hi - lo), 0.0), 1.0)
         assert f[i] == pytest.approx(100.0 ** (-i / 8) * (1.0 - share + share / 4.0))
-    assert amplitude == pytest.approx(1.0 + 0.1 * math.log(4.0)) and 0 < lo < hi < 7
+    assert amplitude == pytest.approx(1.0 + 0.1 * math.log(4.0)) and 0 <= lo < hi < 7
     # attention by hand: one layer, three tokens
     m = attention(4, 2, 6, 0.9, rot(2, 10.0, (2.0, 16, 4.0, 1.0)), softcap=2.0)["mixer"]
     w = {"q": torch.randn(24, 8, generator=g, dtype=torch.float64), "k": torch.randn(12, 8, generator=g, dtype=torch.float64),
